@@ -39,6 +39,7 @@ struct AttnParams {
     const int* block_table;
     int max_pages, page_size, Hq, Hkv, hd, window, BQ, nsplit;
     int hdv;              // width of a value row and of an output row (hd for ordinary attention)
+    int vrow;             // numbers from one value row to the next (hdv; hd where values are the first hdv of the key rows)
     const float* sinks;   // [Hq] or null: exp(sinks[h]) joins the softmax denominator once, with no key and no value
     int v_shared;         // the value rows belong to no kv head: every query reads the whole row of hdv values of a slot
     int out_f32;          // out is float whatever the dtype of q and the caches
@@ -57,7 +58,7 @@ __device__ __forceinline__ void store_out(const AttnParams& p, size_t i, float v
 
 // Where the value row of a slot begins for kv head kvh.
 __device__ __forceinline__ size_t value_row(const AttnParams& p, size_t slot, int kvh) {
-    return p.v_shared ? slot * (size_t)p.hdv : (slot * p.Hkv + kvh) * (size_t)p.hdv;
+    return p.v_shared ? slot * (size_t)p.vrow : (slot * p.Hkv + kvh) * (size_t)p.vrow;
 }
 
 template <typename T>
@@ -316,8 +317,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_kernel(AttnParams p)
     }
     float* myP = Ps + warp * GMAX * 32;
     const size_t row_stride = (size_t)p.Hkv * hd;        // of a key row
-    const size_t vrow_stride = p.v_shared ? (size_t)hdv : (size_t)p.Hkv * hdv;      // of a value row
-    const size_t vhead = p.v_shared ? 0 : (size_t)kvh * hdv;                       // this kv head's place in it
+    const size_t vrow_stride = p.v_shared ? (size_t)p.vrow : (size_t)p.Hkv * p.vrow;      // of a value row
+    const size_t vhead = p.v_shared ? 0 : (size_t)kvh * p.vrow;                    // this kv head's place in it
 
     for (int kb = klo + warp * BK; kb < khi; kb += NWARPS * BK) {
         const int kpos = kb + lane;
@@ -481,7 +482,7 @@ template <typename T>
 bool decode_eligible(const AttnParams& p) {
     const int G = p.Hq / p.Hkv;
     const int gmax = G <= 1 ? 1 : G <= 2 ? 2 : G <= 4 ? 4 : G <= 8 ? 8 : 16;
-    return p.BQ == 1 && G <= 16 && p.hd <= 256 && p.hdv <= 256 && p.hdv % 2 == 0 && (p.hd * sizeof(T)) % 16 == 0 &&
+    return p.BQ == 1 && G <= 16 && p.hd <= 256 && p.hdv <= 256 && p.hdv % 2 == 0 && p.vrow % 2 == 0 && (p.hd * sizeof(T)) % 16 == 0 &&
            ((uintptr_t)p.k_cache % 16 == 0) && ((uintptr_t)p.v_cache % 16 == 0) &&
            decode_smem_bytes(G, gmax, p.hd, p.hdv) <= 48 * 1024;
 }
@@ -560,12 +561,14 @@ LLB_EXPORT long long llb_attention_scratch_floats(int num_tiles, int Hq, int hd,
 // head's softmax weights with the values of ALL kv heads, for mixers that combine heads' weights after the softmax.
 // out_f32 != 0: out is float whatever `dtype` says.
 // softcap > 0: every score (after `scale`) becomes softcap * tanh(score / softcap); sinks are not capped.
-LLB_EXPORT int llb_paged_attention_capped(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
-                                          const int* tile_span, const int* tile_q0, int num_tiles, const int* span_row,
-                                          const int* span_len, const int* span_pos, const int* block_table,
-                                          int max_pages, int page_size, int Hq, int Hkv, int hd, int hdv,
-                                          const float* sinks, int window, float scale, float softcap, int BQ, int nsplit,
-                                          float* scratch, int v_shared, int out_f32, cudaStream_t stream) {
+// vrow: numbers from one (slot, kv head)'s value row to the next; hdv, or hd with v_cache == k_cache: the values are the first
+// hdv numbers of the key rows.
+LLB_EXPORT int llb_paged_attention_rows(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
+                                        const int* tile_span, const int* tile_q0, int num_tiles, const int* span_row,
+                                        const int* span_len, const int* span_pos, const int* block_table,
+                                        int max_pages, int page_size, int Hq, int Hkv, int hd, int hdv, int vrow,
+                                        const float* sinks, int window, float scale, float softcap, int BQ, int nsplit,
+                                        float* scratch, int v_shared, int out_f32, cudaStream_t stream) {
     if (num_tiles == 0) return 0;
     LLB_REQUIRE(num_tiles > 0 && Hq > 0 && Hkv > 0 && hd > 0 && hdv > 0 && page_size > 0 && max_pages > 0 && BQ > 0,
                 "attention: bad sizes");
@@ -580,13 +583,25 @@ LLB_EXPORT int llb_paged_attention_capped(const void* q, const void* k_cache, co
     p.max_pages = max_pages; p.page_size = page_size; p.Hq = Hq; p.Hkv = Hkv; p.hd = hd;
     p.window = window; p.BQ = BQ; p.nsplit = nsplit; p.scale = scale;
     p.softcap = softcap > 0.0f ? softcap : 0.0f;
-    p.hdv = hdv; p.sinks = sinks;
+    p.hdv = hdv; p.vrow = vrow; p.sinks = sinks;
+    LLB_REQUIRE(vrow >= hdv, "attention: value rows of %d numbers, %d apart", hdv, vrow);
     p.v_shared = v_shared ? 1 : 0; p.out_f32 = out_f32 ? 1 : 0;
     p.part_acc = scratch;
     p.part_ml = scratch ? scratch + (size_t)num_tiles * Hq * BQ * nsplit * hdv : nullptr;
     if (dtype == LLB_F32) return launch_attention<float>(p, num_tiles, stream);
     if (dtype == LLB_BF16) return launch_attention<__nv_bfloat16>(p, num_tiles, stream);
     return llb_fail("attention: unknown dtype %d", dtype);
+}
+
+LLB_EXPORT int llb_paged_attention_capped(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
+                                          const int* tile_span, const int* tile_q0, int num_tiles, const int* span_row,
+                                          const int* span_len, const int* span_pos, const int* block_table,
+                                          int max_pages, int page_size, int Hq, int Hkv, int hd, int hdv,
+                                          const float* sinks, int window, float scale, float softcap, int BQ, int nsplit,
+                                          float* scratch, int v_shared, int out_f32, cudaStream_t stream) {
+    return llb_paged_attention_rows(q, k_cache, v_cache, out, dtype, tile_span, tile_q0, num_tiles, span_row, span_len, span_pos,
+                                    block_table, max_pages, page_size, Hq, Hkv, hd, hdv, hdv, sinks, window, scale, softcap, BQ,
+                                    nsplit, scratch, v_shared, out_f32, stream);
 }
 
 LLB_EXPORT int llb_paged_attention_shared(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,

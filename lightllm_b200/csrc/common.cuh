@@ -74,6 +74,14 @@ struct LlbGluArgs {
     int kind;
     float alpha, limit, up_shift;
 };
+// The store epilogue of a contraction takes the same arguments with the kinds of a plain activation (no gate):
+//   LLB_ACT_SQUARED_RELU   max(v, 0)^2          anything else: v
+enum LlbAct { LLB_ACT_SQUARED_RELU = 16 };
+__device__ __forceinline__ float llb_act(float v, int kind) {
+    if (kind != LLB_ACT_SQUARED_RELU) return v;
+    v = fmaxf(v, 0.0f);
+    return v * v;
+}
 static inline LlbGluArgs llb_glu_silu() { return LlbGluArgs{LLB_GLU_SILU, 1.0f, 0.0f, 0.0f}; }
 
 static inline int llb_ceil_div(int a, int b) { return (a + b - 1) / b; }

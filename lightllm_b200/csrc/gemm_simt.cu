@@ -22,8 +22,8 @@ struct Epilogue {
                                                 float* residual, bool has1, const LlbGluArgs& glu) {
         if (EPI == LLB_EPI_STORE) {
             TO* o = (TO*)out + (size_t)m * N + n;
-            o[0] = llb_from_float<TO>(a0);
-            if (has1) o[1] = llb_from_float<TO>(a1);
+            o[0] = llb_from_float<TO>(llb_act(a0, glu.kind));
+            if (has1) o[1] = llb_from_float<TO>(llb_act(a1, glu.kind));
         } else if (EPI == LLB_EPI_STORE_F32) {
             float* o = (float*)out + (size_t)m * N + n;
             o[0] = a0;
@@ -213,7 +213,8 @@ int dispatch_epilogue(int epi, const void* A, const void* W, const void* bias, v
 // A [M,K] (a_dtype), W [N,K] (w_dtype), bias [N] float or null.  `out` is [M,N] of a_dtype
 // (STORE), [M,N] float (STORE_F32) or [M,N/2] of a_dtype (SWIGLU, N even); `residual` is
 // [M,N] float (RESIDUAL).  Supported: (float,float), (bf16,bf16), (bf16 activations, float weights).
-// glu_kind .. glu_up_shift: the gated activation of the GLU epilogue (LLB_GLU_*, see llb_glu).
+// glu_kind .. glu_up_shift: the gated activation of the GLU epilogue (LLB_GLU_*, see llb_glu); under STORE a kind of LlbAct
+// is a plain activation of every output.
 LLB_EXPORT int llb_gemm_simt_glu(const void* A, int a_dtype, const void* W, const void* bias, int w_dtype, void* out,
                                  float* residual, int epilogue, int M, int N, int K, int glu_kind, float glu_alpha,
                                  float glu_limit, float glu_up_shift, cudaStream_t stream) {

@@ -113,6 +113,10 @@ __device__ __forceinline__ void epilogue_row(const GemmParams& p, int m, int nb,
                     if (nb + j + 1 < p.N) o[j >> 1] = __float2bfloat16_rn(glu_pair<false>(p.glu, v[j], v[j + 1]));
             }
         } else if (EPI == LLB_EPI_STORE) {
+            if (p.glu.kind == LLB_ACT_SQUARED_RELU) {
+#pragma unroll
+                for (int j = 0; j < CHUNK; ++j) v[j] = llb_act(v[j], LLB_ACT_SQUARED_RELU);
+            }
             __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)m * p.N + nb;
             if (full && (p.N % 8) == 0) {
 #pragma unroll
@@ -278,7 +282,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                         __float2bfloat16_rn(glu_pair<false>(p.glu, v, other));
                             } else if (m < p.M && n < p.N) {
                                 const size_t idx = (size_t)m * p.N + n;
-                                if (EPI == LLB_EPI_STORE) ((__nv_bfloat16*)p.out)[idx] = __float2bfloat16_rn(v);
+                                if (EPI == LLB_EPI_STORE) ((__nv_bfloat16*)p.out)[idx] = __float2bfloat16_rn(llb_act(v, p.glu.kind));
                                 else if (EPI == LLB_EPI_STORE_F32) ((float*)p.out)[idx] = v;
                                 else if (gridDim.z == 1) p.residual[idx] += v;
                                 else atomicAdd(p.residual + idx, v);
@@ -344,6 +348,10 @@ __device__ __forceinline__ void staged_chunk(const GemmParams& p, const CUtensor
         for (int c = 0; c < 8; ++c)
             *reinterpret_cast<float4*>(row + ((c ^ (lane & 7)) * 16)) = make_float4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
     } else if (EPI == LLB_EPI_STORE) {
+        if (p.glu.kind == LLB_ACT_SQUARED_RELU) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = llb_act(v[j], LLB_ACT_SQUARED_RELU);
+        }
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             uint32_t w[4];
@@ -1002,7 +1010,8 @@ int dispatch_epi(int epi, const CUtensorMap& ma, const CUtensorMap& mb, const Ge
 // whose output row is a multiple of 16 bytes: its pieces add themselves into `residual`, float adds that commute up
 // to rounding, and the meeting place is not touched).  error_flag: one int that the kernel
 // raises if a wait inside it ran out of time (the result is then invalid), or null.
-// glu_kind .. glu_up_shift: the gated activation of the GLU epilogue (LLB_GLU_*, see llb_glu).
+// glu_kind .. glu_up_shift: the gated activation of the GLU epilogue (LLB_GLU_*, see llb_glu); under STORE a kind of LlbAct
+// is a plain activation of every output.
 LLB_EXPORT int llb_gemm_tcgen05_glu(const void* A, const void* W, const float* bias, void* out, float* residual,
                                     int epilogue, int M, int N, int K, int split_k, float* partials, int* counters,
                                     int* error_flag, int glu_kind, float glu_alpha, float glu_limit, float glu_up_shift,

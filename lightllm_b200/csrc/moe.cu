@@ -8,6 +8,9 @@
 // are -1 (every later kernel skips such a pair) and `dense` has `real` columns.  Gate rows: the `n_gate` rows of w behind
 // the E routing rows give sigmoid(w . x) in `gate_out` (a per-token gate on a shared expert), from the same staged row.
 //
+// With an optional bias on the logits, and with a third kind of score: the logit itself, the weights being the softmax over
+// the chosen logits alone (`score` 2).
+//
 // One block per token, a warp an expert's dot product.  The result is written twice: as lists (`ids`, `weights` [T, top], in the order of the choice) and
 // as a dense row of weights over all experts (`dense` [T, E], zero for the experts not chosen), which is what the
 // contraction-shaped expert path multiplies the experts' activations by.
@@ -23,7 +26,8 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const TX* __restrict__ x
                                                         int softmax, int renorm, float scale, int* __restrict__ ids,
                                                         float* __restrict__ weights, float* __restrict__ dense, int real,
                                                         int groups, int keep, float renorm_eps, int n_gate,
-                                                        float* __restrict__ idw, float* __restrict__ gate_out) {
+                                                        float* __restrict__ idw, float* __restrict__ gate_out,
+                                                        const float* __restrict__ bias) {
     extern __shared__ __align__(16) float sm[];  // the token's row [D4], then score [E], choice [E]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
     const int t = blockIdx.x;
@@ -53,13 +57,15 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const TX* __restrict__ x
         }
         const float acc = llb_warp_sum(a0 + a1);
         if (lane == 0) {
-            if (e < E) score[e] = acc;
+            if (e < E) score[e] = bias ? acc + bias[e] : acc;
             else gate_out[(size_t)t * n_gate + (e - E)] = 1.0f / (1.0f + expf(-acc));
         }
     }
     __syncthreads();
     if (warp != 0) return;
-    if (softmax) {
+    if (softmax == 2) {
+        // the logits are the scores; their exponentials are taken once the largest chosen one is known
+    } else if (softmax) {
         float m = -INFINITY;
         for (int e = lane; e < E; e += 32) m = fmaxf(m, score[e]);
         m = llb_warp_max(m);
@@ -94,7 +100,7 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const TX* __restrict__ x
         }
         __syncwarp();
     }
-    float total = 0.0f;
+    float total = 0.0f, first = 0.0f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int arg = E;
@@ -109,7 +115,11 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const TX* __restrict__ x
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
         if (arg >= E) arg = 0;                            // only when every score is NaN
-        const float s = score[arg];
+        float s = score[arg];
+        if (softmax == 2) {                               // the first choice is the largest logit
+            if (k == 0) first = s;
+            s = expf(s - first);
+        }
         total += s;
         if (lane == 0) {
             ids[(size_t)t * top + k] = arg;
@@ -118,7 +128,7 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const TX* __restrict__ x
         }
         __syncwarp();
     }
-    const float mul = renorm ? scale / (total + renorm_eps) : scale;
+    const float mul = renorm || softmax == 2 ? scale / (total + renorm_eps) : scale;
     __syncwarp();
     float mine = 0.0f;
     for (int k = lane; k < top; k += 32) {
@@ -393,10 +403,12 @@ LLB_EXPORT int llb_moe_combine(const float* y, const int* slot, const float* wei
 // `real` on are identity experts (ids -1, their weights summed into idw float [T]).  groups > 1: only experts of the `keep`
 // best of `groups` equal groups of neighbours can be chosen.  n_gate > 0: gate_out float [T, n_gate] = sigmoid of the
 // rows of w behind the routing rows.
-LLB_EXPORT int llb_moe_route_ex(const void* x, int x_dtype, const float* w, const float* correction, int T, int D, int E,
-                                int real, int top, int softmax, int renorm, float renorm_eps, float scale, int groups,
-                                int keep, int n_gate, int* ids, float* weights, float* dense, float* idw, float* gate_out,
-                                cudaStream_t stream) {
+// softmax == 2: the scores are the logits and the weights the softmax over the chosen logits alone.  bias float [E] or null
+// joins the logits (and so choice and weights).
+LLB_EXPORT int llb_moe_route_biased(const void* x, int x_dtype, const float* w, const float* bias, const float* correction,
+                                    int T, int D, int E, int real, int top, int softmax, int renorm, float renorm_eps,
+                                    float scale, int groups, int keep, int n_gate, int* ids, float* weights, float* dense,
+                                    float* idw, float* gate_out, cudaStream_t stream) {
     if (T == 0) return 0;
     LLB_REQUIRE(T > 0 && D > 0 && x && w && ids && weights && dense, "moe_route: bad arguments");
     LLB_REQUIRE(E > 0 && E <= MOE_MAX_EXPERTS && top > 0 && top <= E, "moe_route: top %d of %d experts (at most %d)", top, E,
@@ -417,14 +429,22 @@ LLB_EXPORT int llb_moe_route_ex(const void* x, int x_dtype, const float* w, cons
     if (x_dtype == LLB_F32)
         moe_route_kernel<float><<<blocks, warps * 32, smem, stream>>>((const float*)x, w, correction, T, D, E, top, softmax,
                                                                       renorm, scale, ids, weights, dense, real, groups, keep,
-                                                                      renorm_eps, n_gate, idw, gate_out);
+                                                                      renorm_eps, n_gate, idw, gate_out, bias);
     else if (x_dtype == LLB_BF16)
         moe_route_kernel<__nv_bfloat16><<<blocks, warps * 32, smem, stream>>>(
             (const __nv_bfloat16*)x, w, correction, T, D, E, top, softmax, renorm, scale, ids, weights, dense, real, groups,
-            keep, renorm_eps, n_gate, idw, gate_out);
+            keep, renorm_eps, n_gate, idw, gate_out, bias);
     else
         return llb_fail("moe_route: unknown dtype %d", x_dtype);
     return llb_check_launch("moe_route");
+}
+
+LLB_EXPORT int llb_moe_route_ex(const void* x, int x_dtype, const float* w, const float* correction, int T, int D, int E,
+                                int real, int top, int softmax, int renorm, float renorm_eps, float scale, int groups,
+                                int keep, int n_gate, int* ids, float* weights, float* dense, float* idw, float* gate_out,
+                                cudaStream_t stream) {
+    return llb_moe_route_biased(x, x_dtype, w, nullptr, correction, T, D, E, real, top, softmax, renorm, renorm_eps, scale, groups,
+                                keep, n_gate, ids, weights, dense, idw, gate_out, stream);
 }
 
 LLB_EXPORT int llb_moe_route(const void* x, int x_dtype, const float* w, const float* correction, int T, int D, int E,

@@ -246,14 +246,15 @@ def paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                          num_heads: int, num_kv_heads: int, head_dim: int, window: int, scale: float,
                          bq: int, nsplit: int = 1, scratch: Optional[torch.Tensor] = None,
                          v_head_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
-                         v_shared: bool = False, softcap: float = 0.0) -> None:
+                         v_shared: bool = False, softcap: float = 0.0, v_stride: Optional[int] = None) -> None:
     """Attention of every query row of the listed tiles over its request's pages.  ``v_head_dim``: width of a value
     row (and of an output row) when it differs from the keys'; ``v_cache`` may be ``k_cache`` itself (values read out
     of the key rows).  ``sinks`` float32 [num_heads]: ``exp(sinks[h])`` joins head h's softmax denominator once.
     ``v_shared``: a slot's value row (``v_head_dim`` wide: all kv heads side by side) is read whole by every query head,
     so ``out`` [T, num_heads, v_head_dim] holds each head's weights applied to the values of every kv head.  ``out`` may
     be float32 under bfloat16 inputs.  ``softcap`` > 0: a score becomes ``softcap * tanh(score / softcap)`` (sinks are
-    not capped)."""
+    not capped).  ``v_stride``: numbers from one value row to the next when it is not ``v_head_dim`` (values that are the
+    first ``v_head_dim`` numbers of the key rows: ``head_dim``)."""
     hdv = head_dim if v_head_dim is None else v_head_dim
     if k_cache.dtype != q.dtype or v_cache.dtype != q.dtype or out.dtype not in (q.dtype, torch.float32):
         raise KernelError("attention: q and the caches must share a dtype, out has it or is float32")
@@ -265,12 +266,12 @@ def paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         need = attention_scratch_floats(num_tiles, num_heads, hdv, bq, nsplit)
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"attention: nsplit={nsplit} needs {need} floats of scratch")
-    _check(lib().llb_paged_attention_capped(
+    _check(lib().llb_paged_attention_rows(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _dt(q),
         _i32(tile_span, "tile_span"), _i32(tile_q0, "tile_q0"), num_tiles,
         _i32(span_row, "span_row"), _i32(span_len, "span_len"), _i32(span_pos, "span_pos"),
-        _i32(block_table, "block_table"), max_pages, page_size, num_heads, num_kv_heads, head_dim, hdv, _ptr(sinks),
-        window, ctypes.c_float(scale), ctypes.c_float(softcap or 0.0), bq, nsplit, _ptr(scratch), 1 if v_shared else 0,
+        _i32(block_table, "block_table"), max_pages, page_size, num_heads, num_kv_heads, head_dim, hdv,
+        hdv if v_stride is None else v_stride, _ptr(sinks), window, ctypes.c_float(scale), ctypes.c_float(softcap or 0.0), bq, nsplit, _ptr(scratch), 1 if v_shared else 0,
         1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, _stream()))
 
 
@@ -297,6 +298,7 @@ def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor
 
 
 GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH = 0, 1, 2
+ACT_SQUARED_RELU = 16          # a plain activation of the contractions' STORE epilogue, in the place of a GLU kind
 
 
 def glu_act(x: torch.Tensor, out: torch.Tensor, kind: int, alpha: float = 1.0, limit: float = 0.0,
@@ -537,13 +539,69 @@ def diff_combine(a: torch.Tensor, out: torch.Tensor, num_heads: int, v_head_dim:
                                   ctypes.c_float(eps), ctypes.c_float(mult), _stream()))
 
 
-def head_linear(x: torch.Tensor, x_off: int, w: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t, h, :] = w[h] @ x[t, x_off + h*in : x_off + (h+1)*in] for w [H, out, in]; x [T, C], out [T, H*out]."""
+def head_linear(x: torch.Tensor, x_off: int, w: torch.Tensor, out: torch.Tensor, *, x_head: Optional[int] = None,
+                out_head: Optional[int] = None, rotate=None) -> None:
+    """out[t, h, :on] = w[h] @ x[t, x_off + h * x_head : ... + in] for w [H, on, in]; x [T, C], out [T, H * out_head]; ``x_head``
+    and ``out_head`` are the numbers from head to head (``in`` and ``on`` by default).  ``rotate = (src, dst, dim, positions,
+    inv_freq, interleaved)``: ``dim`` numbers from ``src`` on of a head of x turn by position and go to ``dst`` in the head
+    of out."""
     T, C = x.shape
     H, on, inn = w.shape
-    if x_off < 0 or x_off + H * inn > C or w.dtype != x.dtype or out.dtype != x.dtype or tuple(out.shape) != (T, H * on):
+    x_head, out_head = inn if x_head is None else x_head, on if out_head is None else out_head
+    src, dst, dim, positions, inv_freq, interleaved = rotate if rotate is not None else (0, 0, 0, None, None, False)
+    if x_off < 0 or x_off + H * x_head > C or w.dtype != x.dtype or out.dtype != x.dtype or tuple(out.shape) != (T, H * out_head) \
+            or max(inn, src + dim) > x_head or max(on, dst + dim) > out_head or (dim and inv_freq.numel() != dim // 2):
         raise KernelError(f"head_linear: x {tuple(x.shape)} at {x_off}, w {tuple(w.shape)}, out {tuple(out.shape)}")
-    _check(lib().llb_head_linear(_ptr(x), ctypes.c_longlong(C), x_off, _ptr(w), _ptr(out), _dt(x), T, H, inn, on, _stream()))
+    _check(lib().llb_head_linear_rotated(_ptr(x), ctypes.c_longlong(C), x_off, ctypes.c_longlong(x_head), _ptr(w), _ptr(out),
+                                         ctypes.c_longlong(H * out_head), ctypes.c_longlong(out_head), _dt(x), T, H, inn, on, dim,
+                                         src, dst, 1 if interleaved else 0, _i32(positions, "positions"),
+                                         _f32(inv_freq, "inv_freq"), _stream()))
+
+
+def latent_prepare(src: torch.Tensor, q_off: int, c_off: int, rot_off: int, q_rank: int, rank: int, rot_dim: int,
+                   q_weight: Optional[torch.Tensor], c_weight: torch.Tensor, inv_freq: Optional[torch.Tensor],
+                   interleaved: bool, positions: torch.Tensor, slots: Optional[torch.Tensor], q_out: Optional[torch.Tensor],
+                   cache: Optional[torch.Tensor], eps: float) -> None:
+    """The norms between the projections of attention over a rotated latent (csrc/latent_attention.cu): ``q_out`` [T, q_rank]
+    = rms(src[:, q_off:]) * q_weight; cache rows ``slots`` of ``cache`` [slots, 1, rank + rot_dim] = [rms(src[:, c_off:]) *
+    c_weight | src[:, rot_off:] rotated by position].  ``q_out`` or ``cache`` may be None."""
+    T, C = src.shape
+    if c_off + rank > C or rot_off + rot_dim > C or (q_out is not None and (q_off + q_rank > C or tuple(q_out.shape) != (T, q_rank)
+                                                                             or q_out.dtype != src.dtype)):
+        raise KernelError("latent_prepare: columns or outputs do not fit")
+    if cache is not None and (cache.shape[-1] != rank + rot_dim or cache.dtype != src.dtype or slots.numel() != T):
+        raise KernelError("latent_prepare: the cache plane does not fit")
+    _check(lib().llb_latent_prepare(_ptr(src), _dt(src), ctypes.c_longlong(C), q_off, c_off, rot_off, T, q_rank, rank, rot_dim,
+                                    1 if interleaved else 0, _f32(q_weight, "q_weight"), _f32(c_weight, "c_weight"),
+                                    _f32(inv_freq, "inv_freq"), _i32(positions, "positions"), _i32(slots, "slots"),
+                                    _ptr(q_out), _ptr(cache), ctypes.c_float(eps), _stream()))
+
+
+LATENT_MAX_SPLITS = 8
+
+
+def latent_attention_supports(width: int, rank: int) -> bool:
+    return bool(lib().llb_latent_attention_supports(width, rank))
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, span_row: torch.Tensor, span_len: torch.Tensor,
+                     span_pos: torch.Tensor, num_spans: int, block_table: torch.Tensor, max_pages: int, page_size: int,
+                     num_heads: int, width: int, rank: int, window: int, scale: float, single: bool, nsplit: int = 1,
+                     sinks: Optional[torch.Tensor] = None) -> None:
+    """Attention of every head over key rows of ``width`` numbers whose first ``rank`` are the values (bfloat16; the cache
+    [slots, 1, width]); q [T, H * width], out [T, H * rank].  ``single``: every span is one token; then ``nsplit`` (at most
+    8) pieces of the keys run side by side and are merged inside the kernel."""
+    T = q.shape[0]
+    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+        raise KernelError("latent_attention takes bfloat16")
+    if q.numel() != T * num_heads * width or out.numel() != T * num_heads * rank or cache.shape[-1] != width:
+        raise KernelError("latent_attention: sizes do not fit")
+    if sinks is not None and sinks.numel() != num_heads:
+        raise KernelError(f"latent_attention: sinks must be float32 [{num_heads}]")
+    _check(lib().llb_latent_attention(_ptr(q), _ptr(cache), _ptr(out), T, _i32(span_row, "span_row"), _i32(span_len, "span_len"),
+                                      _i32(span_pos, "span_pos"), num_spans, _i32(block_table, "block_table"), max_pages,
+                                      page_size, num_heads, width, rank, window, ctypes.c_float(scale), 1 if single else 0,
+                                      nsplit, _f32(sinks, "sinks"), _stream()))
 
 
 def retention(src: torch.Tensor, q_off: int, k_off: int, v_off: int, span_row: torch.Tensor, span_len: torch.Tensor,
@@ -665,6 +723,97 @@ def conv_tail_update(src: torch.Tensor, c0: int, channels: int, taps: int, ctx_s
                                       ctypes.c_longlong(tail_off), _stream()))
 
 
+def conv_act(src: torch.Tensor, c0: int, channels: int, weight: torch.Tensor, bias: Optional[torch.Tensor], act, ctx_spans, state,
+             tail_off: int, out: torch.Tensor, fuse_tail: bool = False) -> None:
+    """The causal convolution of :func:`conv_prepare` with a bias and an activation (``None`` or ``"silu"``) on all channels alike,
+    into ``out`` [T, channels] (the dtype of ``src``); tails as there."""
+    T, C = src.shape
+    taps = weight.shape[1]
+    if weight.dtype != torch.float32 or weight.shape[0] != channels or c0 + channels > C or tuple(out.shape) != (T, channels) \
+            or out.dtype != src.dtype or (bias is not None and bias.numel() != channels):
+        raise KernelError(f"conv_act: weight {weight.dtype} {tuple(weight.shape)} for {channels} channels of {C} columns")
+    span_row, _, span_pos, span_slot, num_spans = ctx_spans
+    base, stride = (None, 0) if state is None else _state_base(state)
+    if state is not None and tail_off + (taps - 1) * channels > stride:
+        raise KernelError("conv_act: the tail does not fit in a state slot")
+    _check(lib().llb_conv_act(_ptr(src), _dt(src), ctypes.c_longlong(C), c0, channels, taps, T, _ptr(weight), _f32(bias, "bias"),
+                              {None: 0, "silu": 1}[act], _i32(span_row, "span_row"), _i32(span_pos, "span_pos"),
+                              _i32(span_slot, "span_slot"), num_spans, base, ctypes.c_longlong(stride),
+                              ctypes.c_longlong(tail_off), _ptr(out), 1 if fuse_tail else 0, _stream()))
+
+
+def norm_shift(x: torch.Tensor, w1: torch.Tensor, mix: torch.Tensor, eps: float, ctx_spans, state: torch.Tensor, state_off: int,
+               out1: torch.Tensor, w2: Optional[torch.Tensor] = None, out2: Optional[torch.Tensor] = None,
+               clear: Optional[torch.Tensor] = None) -> None:
+    """RMS norm of the rows of x (float32 [T, D]) by ``w1``, then a shift towards the row before, ``h + (h_before - h) * mix``,
+    into ``out1``; with ``w2`` the norm by another weight into ``out2`` as well; ``clear`` (float32 [T, D]) is zeroed on the
+    way.  A request's last h (float32, D numbers) lies ``state_off`` floats into its slot of ``state``."""
+    T, D = x.shape
+    span_row, span_len, span_pos, span_slot, num_spans = ctx_spans
+    base, stride = _state_base(state)
+    if state_off + D > stride or w1.numel() != D or mix.numel() != D or tuple(out1.shape) != (T, D) or \
+            (w2 is not None and (w2.numel() != D or out2 is None or out2.shape != out1.shape or out2.dtype != out1.dtype)) or \
+            (clear is not None and (clear.dtype != torch.float32 or clear.shape != x.shape)):
+        raise KernelError("norm_shift: sizes do not fit")
+    _check(lib().llb_norm_shift(_f32(x, "x"), _f32(w1, "w1"), _f32(mix, "mix"), _f32(w2, "w2"), _ptr(out1), _ptr(out2), _dt(out1),
+                                _ptr(clear), T, D, ctypes.c_float(eps), _i32(span_row, "span_row"), _i32(span_len, "span_len"),
+                                _i32(span_pos, "span_pos"), _i32(span_slot, "span_slot"), num_spans, base,
+                                ctypes.c_longlong(stride), ctypes.c_longlong(state_off), _stream()))
+
+
+def state_space_chunks_support(state: int, vdim: int, stride: int, x_off: int, b_off: int, c_off: int) -> bool:
+    return bool(lib().llb_state_space_chunks_support(state, vdim, stride, x_off, b_off, c_off))
+
+
+def state_space(xbc: torch.Tensor, x_off: int, b_off: int, c_off: int, dt: torch.Tensor, dt_bias: torch.Tensor,
+                rate: torch.Tensor, skip: torch.Tensor, ctx_spans, num_heads: int, groups: int, state_dim: int, v_head_dim: int,
+                state: torch.Tensor, state_off: int, out: torch.Tensor, single: bool = False, pieces=None) -> None:
+    """The state-space recurrence of Mamba-2 over every span (csrc/state_space.cu).  ``xbc`` [T, C] holds x [H, vdim], B and C
+    [G, N] in columns; ``dt`` a [T, H] view (rows may be strided) before ``dt_bias`` and the softplus; rate = exp(A_log), skip
+    = D, float32 [H]; the state [H, N, vdim] of a request lies ``state_off`` floats into its slot of ``state``; out float32
+    [T, H * vdim].  ``single``: every span is one token.  ``pieces = (item_span, item_c, span_first, num_items, chunk)`` as
+    :func:`retention` takes them asks for the tensor-core kernels (see :func:`state_space_chunks_support`), ``chunk`` a
+    multiple of 64; without it the spans are walked token by token."""
+    T, C = xbc.shape
+    H, G, N, vd = num_heads, groups, state_dim, v_head_dim
+    if x_off + H * vd > C or max(b_off, c_off) + G * N > C:
+        raise KernelError("state_space: x, B or C lie outside the columns")
+    if dt.dim() != 2 or tuple(dt.shape) != (T, H) or dt.stride(1) != 1 or not dt.is_cuda:
+        raise KernelError(f"state_space: dt must be [{T}, {H}] with unit inner stride")
+    if out.dtype != torch.float32 or out.numel() != T * H * vd or any(v.numel() != H for v in (dt_bias, rate, skip)):
+        raise KernelError("state_space: sizes do not fit")
+    span_row, span_len, span_pos, span_slot, num_spans = ctx_spans
+    base, stride = _state_base(state)
+    if state_off + H * N * vd > stride:
+        raise KernelError("state_space: the state does not fit in a slot")
+    item_span = item_c = first = scratch = keep = None
+    items, chunk, multi = 0, 0, False
+    if pieces is not None:
+        item_span, item_c, first, items, chunk = pieces
+        multi = items > num_spans
+        if multi:
+            scratch = torch.empty(items * H * N * vd, dtype=torch.float32, device=xbc.device)
+            keep = torch.empty(items * H, dtype=torch.float32, device=xbc.device)
+    _check(lib().llb_state_space(_ptr(xbc), _dt(xbc), ctypes.c_longlong(C), x_off, b_off, c_off, ctypes.c_void_p(dt.data_ptr()),
+                                 _dt(dt), ctypes.c_longlong(dt.stride(0)), 0, _f32(dt_bias, "dt_bias"), _f32(rate, "rate"),
+                                 _f32(skip, "skip"), _i32(span_row, "span_row"), _i32(span_len, "span_len"),
+                                 _i32(span_pos, "span_pos"), _i32(span_slot, "span_slot"), num_spans, H, G, N, vd, base,
+                                 ctypes.c_longlong(stride), ctypes.c_longlong(state_off), _ptr(out), 1 if single else 0,
+                                 _i32(item_span, "item_span"), _i32(item_c, "item_c"), _i32(first, "span_first"), items, chunk,
+                                 1 if multi else 0, _ptr(scratch), _ptr(keep), _stream()))
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, out: torch.Tensor) -> None:
+    """out = rms(y * silu(z)) * weight with the root mean square of each of ``parts`` equal parts of a row: y float32 [T, n], z a
+    [T, n] view (rows may be strided) in the dtype of out."""
+    T, n = out.shape
+    if y.dtype != torch.float32 or y.numel() != T * n or tuple(z.shape) != (T, n) or z.stride(1) != 1 or z.dtype != out.dtype \
+            or n % parts or weight.numel() != n or not z.is_cuda:
+        raise KernelError("gated_group_norm: sizes do not fit")
+    _check(lib().llb_gated_group_norm(_ptr(y), ctypes.c_void_p(z.data_ptr()), _dt(out), ctypes.c_longlong(z.stride(0)),
+                                      _f32(weight, "weight"), _ptr(out), T, n // parts, parts, ctypes.c_float(eps), _stream()))
+
+
 def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, ctx_spans,
                num_heads: int, num_qk_heads: int, head_dim: int, v_head_dim: int, state: torch.Tensor, state_off: int,
                out: torch.Tensor, blocked: bool = False) -> None:
@@ -717,8 +866,8 @@ def low_rank_up(x: torch.Tensor, x_off: int, w: torch.Tensor, out: torch.Tensor,
 
 
 def moe_route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tensor], top: int, scale: float,
-              ids: torch.Tensor, weights: torch.Tensor, dense: torch.Tensor, softmax: bool = False,
-              renormalize: bool = False, *, renorm_eps: float = 0.0, real: Optional[int] = None, groups: int = 0,
+              ids: torch.Tensor, weights: torch.Tensor, dense: torch.Tensor, softmax=False,
+              renormalize: bool = False, *, bias: Optional[torch.Tensor] = None, renorm_eps: float = 0.0, real: Optional[int] = None, groups: int = 0,
               keep: int = 0, identity_weight: Optional[torch.Tensor] = None, gate_rows: int = 0,
               gate_out: Optional[torch.Tensor] = None) -> None:
     """Routing in float (csrc/moe.cu): x [T, D], w float32 [E + gate_rows, D], correction float32 [E] or None (joins the
@@ -726,7 +875,9 @@ def moe_route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tenso
     ``real`` < E: the router's outputs from ``real`` on are identity experts; their entries of ``ids`` are -1 and a
     token's weights on them are summed into ``identity_weight`` float32 [T].  ``groups`` > 1: only experts of the ``keep``
     best of ``groups`` equal groups of neighbours can be chosen (a group's score is its largest choice score).
-    ``gate_rows``: that many further rows of w give ``gate_out`` float32 [T, gate_rows] = sigmoid(w . x)."""
+    ``gate_rows``: that many further rows of w give ``gate_out`` float32 [T, gate_rows] = sigmoid(w . x).  ``softmax``: False
+    (a sigmoid of each logit), True (over all outputs) or ``"chosen"`` (the logits choose, the weights are the softmax over the
+    chosen logits alone).  ``bias`` float32 [E] joins the logits."""
     T, D = x.shape
     E = w.shape[0] - gate_rows
     real = E if real is None else real
@@ -738,11 +889,13 @@ def moe_route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tenso
         raise KernelError("moe_route: identity experts need identity_weight float32 [T]")
     if gate_rows and (gate_out is None or gate_out.numel() != T * gate_rows):
         raise KernelError("moe_route: gate rows need gate_out float32 [T, gate_rows]")
-    _check(lib().llb_moe_route_ex(_ptr(x), _dt(x), _f32(w, "w"), _f32(correction, "correction"), T, D, E, real, top,
-                                  1 if softmax else 0, 1 if renormalize else 0, ctypes.c_float(renorm_eps),
-                                  ctypes.c_float(scale), groups, keep, gate_rows, _i32(ids, "ids"), _f32(weights, "weights"),
-                                  _f32(dense, "dense"), _f32(identity_weight, "identity_weight"), _f32(gate_out, "gate_out"),
-                                  _stream()))
+    if bias is not None and bias.numel() != E:
+        raise KernelError(f"moe_route: the bias must be float32 [{E}]")
+    _check(lib().llb_moe_route_biased(_ptr(x), _dt(x), _f32(w, "w"), _f32(bias, "bias"), _f32(correction, "correction"), T, D, E, real,
+                                      top, 2 if softmax == "chosen" else 1 if softmax else 0, 1 if renormalize else 0,
+                                      ctypes.c_float(renorm_eps), ctypes.c_float(scale), groups, keep, gate_rows,
+                                      _i32(ids, "ids"), _f32(weights, "weights"), _f32(dense, "dense"),
+                                      _f32(identity_weight, "identity_weight"), _f32(gate_out, "gate_out"), _stream()))
 
 
 def moe_scale(act: torch.Tensor, dense: torch.Tensor, num_experts: int, width: int) -> None:

@@ -298,3 +298,169 @@ LLB_EXPORT int llb_conv_tail_update(const void* src, int src_dtype, long long ro
     else return llb_fail("conv_tail_update: unknown dtype %d", src_dtype);
     return llb_check_launch("conv_tail_update");
 }
+
+// ---------------------------------------------------------------------------------------------------------------------
+// The convolution alone, with a bias and an activation, for many channels that are not heads yet: a thread owns V
+// neighbouring channels over a run of ROWS rows of the step and carries the last taps - 1 inputs in registers, so that
+// every input is read once (four channels at a time where they are aligned).  Rows may cross spans: at a span's first row the carried inputs are the
+// request's tail.
+namespace {
+
+struct ConvActParams {
+    const void* src;             // [T, row_stride]; channels in columns c0 .. c0 + C - 1
+    long long row_stride;
+    int c0, C, taps, T, num_spans, act;
+    const float* w;              // [C, taps]
+    const float* bias;           // [C] or null
+    const int* span_row;
+    const int* span_pos;
+    const int* span_slot;
+    float* state;
+    long long state_stride, tail_off;
+    void* out;                   // [T, C], the dtype of src
+    int fuse_tail;
+};
+
+template <typename T, int V> struct ConvVec;
+template <typename T> struct ConvVec<T, 1> {
+    static __device__ __forceinline__ void load(const T* p, float (&v)[1]) { v[0] = llb_to_float(*p); }
+    static __device__ __forceinline__ void store(T* p, const float (&v)[1]) { *p = llb_from_float<T>(v[0]); }
+};
+template <> struct ConvVec<float, 4> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+        const float4 q = *reinterpret_cast<const float4*>(p);
+        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+    }
+    static __device__ __forceinline__ void store(float* p, const float (&v)[4]) {
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+};
+template <> struct ConvVec<__nv_bfloat16, 4> {
+    static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[4]) {
+        const uint2 q = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+        v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+    }
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[4]) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    }
+};
+
+// TAPS: the most taps this instantiation carries (a smaller `taps` leaves its first slots unused).
+template <typename T, int V, int TAPS, int ROWS>
+__global__ void __launch_bounds__(128) conv_act_kernel(ConvActParams p) {
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (c >= p.C) return;
+    const int t0 = blockIdx.y * ROWS, t1 = min(p.T, t0 + ROWS);
+    const T* src = (const T*)p.src + p.c0 + c;
+    const int taps = p.taps, skip = TAPS - taps;           // weight j of the channel sits in slot skip + j
+    float w[TAPS][V], b[V];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int i = 0; i < V; ++i) w[j][i] = j >= skip ? p.w[(size_t)(c + i) * taps + (j - skip)] : 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) b[i] = p.bias ? p.bias[c + i] : 0.0f;
+    int span = span_of_row(p.span_row, p.num_spans, t0);
+    int next = span + 1 < p.num_spans ? p.span_row[span + 1] : p.T;      // first row of the span after this one
+    float u[TAPS][V];                                      // slot TAPS - 1: the current row; slot TAPS - 1 - m: m rows before
+    // the inputs before row t (local rows into its span), from this step's rows or from the request's tail
+    auto reload = [&](int t, int local) {
+        const int pos = p.span_pos[span] + local;
+        const float* tail = p.state + (long long)p.span_slot[span] * p.state_stride + p.tail_off;
+#pragma unroll
+        for (int m = 1; m < TAPS; ++m) {
+            float v[V];
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] = 0.0f;
+            if (m < taps) {
+                if (local - m >= 0) {
+                    ConvVec<T, V>::load(src + (long long)(t - m) * p.row_stride, v);
+                } else if (pos - m >= 0) {
+#pragma unroll
+                    for (int i = 0; i < V; ++i) v[i] = tail[(size_t)(taps - 1 + local - m) * p.C + c + i];
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < V; ++i) u[TAPS - 1 - m][i] = v[i];
+        }
+    };
+    reload(t0, t0 - p.span_row[span]);
+    T* out = (T*)p.out + c;
+    for (int t = t0; t < t1; ++t) {
+        if (t == next) {
+            ++span;
+            next = span + 1 < p.num_spans ? p.span_row[span + 1] : p.T;
+            reload(t, 0);
+        }
+        ConvVec<T, V>::load(src + (long long)t * p.row_stride, u[TAPS - 1]);
+        float y[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            float a = b[i];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) a = fmaf(w[j][i], u[j][i], a);
+            y[i] = p.act == 1 ? llb_silu(a) : a;
+        }
+        ConvVec<T, V>::store(out + (size_t)t * p.C, y);
+        if (p.fuse_tail) {                                  // (the span is this one row: the carried inputs are its new tail)
+            float* tail = p.state + (long long)p.span_slot[span] * p.state_stride + p.tail_off;
+#pragma unroll
+            for (int m = 0; m < TAPS - 1; ++m)
+                if (m < taps - 1)
+#pragma unroll
+                    for (int i = 0; i < V; ++i) tail[(size_t)(taps - 2 - m) * p.C + c + i] = u[TAPS - 1 - m][i];
+        }
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+            for (int i = 0; i < V; ++i) u[j][i] = u[j + 1][i];
+    }
+}
+
+template <typename T, int V, int TAPS>
+int launch_conv_act_rows(const ConvActParams& p, cudaStream_t stream) {
+    const int groups = (p.C + V - 1) / V;
+    const unsigned gx = (unsigned)((groups + 127) / 128);
+    if ((long long)gx * p.T <= 148 * 8 || p.fuse_tail)
+        conv_act_kernel<T, V, TAPS, 1><<<dim3(gx, p.T), 128, 0, stream>>>(p);
+    else if ((long long)gx * p.T <= 148 * 32)
+        conv_act_kernel<T, V, TAPS, 4><<<dim3(gx, (p.T + 3) / 4), 128, 0, stream>>>(p);
+    else
+        conv_act_kernel<T, V, TAPS, 16><<<dim3(gx, (p.T + 15) / 16), 128, 0, stream>>>(p);
+    return llb_check_launch("conv_act");
+}
+
+template <typename T>
+int launch_conv_act(const ConvActParams& p, cudaStream_t stream) {
+    constexpr int bytes = 4 * sizeof(T);
+    const bool vec = p.C % 4 == 0 && p.c0 % 4 == 0 && p.row_stride % 4 == 0 && (uintptr_t)p.src % bytes == 0 && (uintptr_t)p.out % bytes == 0;
+    if (p.taps <= 4) return vec ? launch_conv_act_rows<T, 4, 4>(p, stream) : launch_conv_act_rows<T, 1, 4>(p, stream);
+    return vec ? launch_conv_act_rows<T, 4, CONV_MAX_TAPS>(p, stream) : launch_conv_act_rows<T, 1, CONV_MAX_TAPS>(p, stream);
+}
+
+}  // namespace
+
+// src [T, row_stride] (dtype) holds C channels from column c0 on; w float [C, taps], bias float [C] or null, act 0 none or
+// 1 SiLU; out [T, C] (dtype).  Spans, state and tails as llb_conv_prepare; fuse_tail != 0 only when every span is one
+// token (else llb_conv_tail_update afterwards).
+LLB_EXPORT int llb_conv_act(const void* src, int dtype, long long row_stride, int c0, int C, int taps, int T, const float* w,
+                            const float* bias, int act, const int* span_row, const int* span_pos, const int* span_slot,
+                            int num_spans, float* state, long long state_stride, long long tail_off, void* out, int fuse_tail,
+                            cudaStream_t stream) {
+    if (T == 0) return 0;
+    LLB_REQUIRE(T > 0 && C > 0 && src && w && out && span_row && span_pos && span_slot && num_spans > 0, "conv_act: bad arguments");
+    LLB_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, "conv_act: %d taps; at most %d", taps, CONV_MAX_TAPS);
+    LLB_REQUIRE(taps == 1 || state != nullptr, "conv_act: a convolution of %d taps needs the requests' state", taps);
+    LLB_REQUIRE(!fuse_tail || T == num_spans, "conv_act: the tail is only written here when every span is one token");
+    LLB_REQUIRE(T <= 65535 * 16, "conv_act: too many rows");
+    ConvActParams p;
+    p.src = src; p.row_stride = row_stride; p.c0 = c0; p.C = C; p.taps = taps; p.T = T; p.num_spans = num_spans; p.act = act;
+    p.w = w; p.bias = bias; p.span_row = span_row; p.span_pos = span_pos; p.span_slot = span_slot; p.state = state;
+    p.state_stride = state_stride; p.tail_off = tail_off; p.out = out; p.fuse_tail = taps > 1 ? fuse_tail : 0;
+    if (dtype == LLB_F32) return launch_conv_act<float>(p, stream);
+    if (dtype == LLB_BF16) return launch_conv_act<__nv_bfloat16>(p, stream);
+    return llb_fail("conv_act: unknown dtype %d", dtype);
+}

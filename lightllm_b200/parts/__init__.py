@@ -8,15 +8,17 @@ from .differential_attention import DifferentialAttentionMixer
 from .sink_attention import KeyValuedAttentionMixer
 from .moe import RoutedExperts
 from .stream import StreamReinjection, StreamStepVector
-from .input_conv import CausalInputConv
+from .input_conv import CausalInputConv, TokenShift
 from .mixed_heads_attention import MixedHeadsAttention
 from .matrix_memory import MatrixMemoryMixer
 from .joined_mixers import JoinedMixers
 from .embedding import LMHead, TokenEmbedding
 from .gated_attention import GatedAttentionMixer, LatentAttentionMixer
-from .mlp import GatedMLP
+from .mlp import GatedMLP, PlainMLP
 from .norm import LayerNorm, RMSNorm
 from .retention import RetentionMixer
+from .rotary_latent_attention import RotaryLatentAttentionMixer
+from .state_space import StateSpaceMixer
 from .rotary import NoPositionEncoding, RotaryEmbedding
 
 __all__ = ["CacheView", "FeedForward", "Mixer", "Norm", "Part", "PositionEncoding", "AttentionMixer", "Block",
@@ -24,4 +26,4 @@ __all__ = ["CacheView", "FeedForward", "Mixer", "Norm", "Part", "PositionEncodin
            "LatentAttentionMixer", "RetentionMixer", "NoPositionEncoding", "RotaryEmbedding", "ConvAttentionMixer",
            "ChannelDeltaMixer", "RoutedExperts", "StreamReinjection", "StreamStepVector", "CausalInputConv",
            "MixedHeadsAttention", "MatrixMemoryMixer", "JoinedMixers", "DifferentialAttentionMixer",
-           "KeyValuedAttentionMixer"]
+           "KeyValuedAttentionMixer", "TokenShift", "PlainMLP", "RotaryLatentAttentionMixer", "StateSpaceMixer"]

@@ -61,7 +61,7 @@ class AttentionMixer(Mixer):
         self.qkv_bias, self.out_bias = qkv_bias, out_bias
         # Values may be narrower or wider than keys; ``sinks`` (float32 [heads], set by mixers that have them) adds
         # exp(sink_h) to each head's softmax denominator; ``values_in_keys``: the cache keeps no value rows and the
-        # kernels read the values out of the key rows.  Any of these takes the CUDA-core attention kernels.
+        # kernels read the values out of the key rows (the first v_head_dim numbers of each).  Any of these takes the CUDA-core attention kernels.
         self.v_head_dim = head_dim if v_head_dim is None else int(v_head_dim)
         self.sinks: Optional[torch.Tensor] = None
         self.values_in_keys = False
@@ -369,7 +369,8 @@ class AttentionMixer(Mixer):
                                   dtype=torch.float32, device=q.device)
         ops.paged_attention_simt(q, cache.k, cache.k if self.values_in_keys else cache.v, out, tile_span, tile_q0, ntiles,
                                  *common, bq, nsplit, scratch, v_head_dim=hdv, sinks=self.sinks,
-                                 v_shared=self.value_cross > 1, softcap=self.softcap or 0.0)
+                                 v_shared=self.value_cross > 1, softcap=self.softcap or 0.0,
+                                 v_stride=self.head_dim if self.values_in_keys else None)
 
 
 register_part("mixer", "attention", AttentionMixer)

@@ -19,7 +19,8 @@ Roles and what each must provide:
 ``embedding``  ``forward(token_ids[T] int32, ctx) -> residual[T, D] float32``.
 ``head``       ``forward(x[R, D], ctx) -> logits[R, V] float32``.
 ``filter``     ``forward(h[T, D] float32, ctx, cache, out_dtype, last_reader) -> x[T, D]``: what a sub-block reads instead
-               of h; ``state_floats()`` floats of the run's state plane are its own.
+               of h; ``state_floats()`` floats of the run's state plane are its own.  A filter may take the norm
+               before it into its own kernel (``takes_norm``, ``forward_normed``).
 ``stream``     ``forward(residual, ctx)``: rewrites the stream before a run entry.
 
 The residual stream is float32 in both precisions, so the residual sum is exact to float.

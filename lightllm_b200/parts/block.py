@@ -168,10 +168,35 @@ class Block(Part):
         return sb.filter.forward(h, ctx, view, ctx.dtype if ctx is not None and ctx.dtype is not None else h.dtype,
                                  last_reader=sb.last_reader)
 
+    def _fused_inputs(self, residual, ctx, cache, into):
+        """The inputs of a parallel layer's sub-blocks from one kernel, or None: the first sub-block's filter takes the norm
+        before it into its own kernel, with the norm of the one other sub-block if there is one (see
+        :meth:`~.input_conv.TokenShift.takes_norm`), and clears ``into``."""
+        first, rest = self.subs[0], self.subs[1:]
+        takes = getattr(first.filter, "takes_norm", None)
+        if takes is None or any(sb.filter is not None or sb.norm_before is None or sb.shares_input_of is not None for sb in rest) or \
+                not takes(first.norm_before, [sb.norm_before for sb in rest]):
+            return None
+        dtype = ctx.dtype if ctx is not None and ctx.dtype is not None else residual.dtype
+        x, others = first.filter.forward_normed(residual, first.norm_before, [sb.norm_before for sb in rest], ctx,
+                                                cache.at(first.filter_offset, pages=False), dtype, clear=into)
+        return [x, *others]
+
     def forward(self, residual, ctx, cache) -> None:
         scaled = self.branch_scale != 1.0
-        into = torch.zeros_like(residual) if scaled else None          # the branches' sum, scaled as it joins the stream
+        into = None          # the branches' sum, scaled as it joins the stream
         normed: Dict[int, torch.Tensor] = {}
+        if self.arrangement == "parallel" and self.filtered:
+            into = torch.empty_like(residual) if scaled else None
+            inputs = self._fused_inputs(residual, ctx, cache, into)
+            if inputs is not None:
+                for sb, x in zip(self.subs, inputs):
+                    self._run(sb, x, residual, ctx, cache, into)
+                if scaled:
+                    ops.axpy(into, residual, self.branch_scale)
+                return
+        if scaled:
+            into = into.zero_() if into is not None else torch.zeros_like(residual)
         if self.arrangement == "parallel":
             # every branch reads the same h, so all inputs are computed before anything is added
             inputs = [self._filtered_input(i, residual, ctx, cache, normed) if sb.filter is not None

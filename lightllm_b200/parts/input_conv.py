@@ -1,4 +1,4 @@
-"""A causal convolution over time on what a sub-block reads."""
+"""Filters over time on what a sub-block reads: a causal convolution, a shift towards the token before."""
 from __future__ import annotations
 
 from typing import List, Optional
@@ -64,4 +64,46 @@ class CausalInputConv(InputFilter):
         return out
 
 
+class TokenShift(CausalInputConv):
+    """``x_t = h_t + (h_(t-1) - h_t) * mix`` on every channel of the normed stream h, zeros before the sequence's first token: a
+    convolution of the two taps ``mix`` and ``1 - mix``.  ``weight_name`` is ``[channels]``.
+
+    A request's last row of h lives in the run's state plane (float32).  Where the norm before it is an RMS norm, the filter
+    takes it into a kernel of its own (:meth:`forward_normed`), together with the norm that another branch of a parallel layer
+    takes of the same stream: the rows are read once for all of them."""
+
+    def __init__(self, prefix: str, channels: int, weight_name: str = "weight"):
+        super().__init__(prefix, channels, 2, weight_name, residual=False)
+        self.mix = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [WeightSpec(self.name, (self.channels,), init=("normal", 0.3))]
+
+    def bind(self, tensors, dtype, device) -> None:
+        self.mix = tensors[self.name].float().contiguous()
+        self.weight = torch.stack([self.mix, 1.0 - self.mix], dim=1).contiguous()
+
+    def takes_norm(self, norm, others=()) -> bool:
+        """Whether :meth:`forward_normed` computes ``norm`` (and the ``others`` of the same stream, at most one) itself: RMS
+        norms with one eps between them and float32 weights."""
+        def rms(n):
+            f = getattr(n, "rms_parameters", None)
+            return f() if f is not None else None
+        first = rms(norm)
+        rest = [rms(n) for n in others]
+        return (first is not None and first[0] is not None and first[0].dtype == torch.float32 and len(rest) <= 1
+                and all(o is not None and o[0].dtype == torch.float32 and o[1] == first[1] for o in rest))
+
+    def forward_normed(self, residual, norm, others, ctx, cache: CacheView, out_dtype, clear=None):
+        """(the shifted normed stream, [the ``others``' normed streams]) of the float32 stream; ``clear`` (float32, the stream's
+        shape) is zeroed by the same kernel."""
+        w1, eps = norm.rms_parameters()
+        w2 = others[0].rms_parameters()[0] if others else None
+        out = torch.empty(residual.shape, dtype=out_dtype, device=residual.device)
+        out2 = torch.empty_like(out) if others else None
+        ops.norm_shift(residual, w1, self.mix, eps, span_arrays(ctx), cache.state, cache.state_offset, out, w2, out2, clear)
+        return out, [out2] if others else []
+
+
 register_part("filter", "causal_conv", CausalInputConv)
+register_part("filter", "token_shift", TokenShift)

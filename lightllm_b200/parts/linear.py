@@ -93,7 +93,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
            out: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None, glu=None) -> Optional[torch.Tensor]:
     """Run the contraction; returns ``out`` (allocated here when not given), or ``None`` for the
     residual epilogue, which adds into ``residual``.  ``glu = (kind, alpha, limit, up_shift)``: the gated activation
-    of the SWIGLU epilogue when it is not SiLU (``ops.glu_act`` has the kinds)."""
+    of the SWIGLU epilogue when it is not SiLU (``ops.glu_act`` has the kinds); under STORE a plain activation of every output
+    (``ops.ACT_SQUARED_RELU``)."""
     M, N = x.shape[0], w.shape[0]
     if epilogue != RESIDUAL and out is None:
         cols = N // 2 if epilogue == SWIGLU else N

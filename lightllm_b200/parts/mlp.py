@@ -6,6 +6,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..config import register_part
+from ..csrc import ops
 from ..weights import WeightSpec
 from . import linear as L
 from .base import FeedForward, LazyNorm
@@ -84,4 +85,38 @@ class GatedMLP(FeedForward):
         L.linear(act, self.w_down, self.b_down, L.RESIDUAL, residual=residual)
 
 
+# activation name of a feed-forward without a gate -> the code of the contractions' store epilogue
+PLAIN_ACTIVATIONS = {"squared_relu": ops.ACT_SQUARED_RELU}
+
+
+class PlainMLP(FeedForward):
+    """A feed-forward without a gate, ``h += act(x Wu^T) Wd^T``; ``squared_relu``: ``max(z, 0)^2``.  The activation is taken in the
+    epilogue of the first contraction, from its float accumulators; no biases."""
+
+    graph_safe = True
+
+    def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, activation: str = "squared_relu",
+                 names: Optional[Dict[str, str]] = None, weight_suffix: str = ".weight"):
+        if activation not in PLAIN_ACTIVATIONS:
+            raise ValueError(f"the plain feed-forward implements {sorted(PLAIN_ACTIVATIONS)}, not {activation!r}")
+        self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
+        names = {"up": "up_proj", "down": "down_proj", **(names or {})}
+        self.up_name, self.down_name = (f"{prefix}.{names[n]}{weight_suffix}" for n in ("up", "down"))
+        self.w_up = self.w_down = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        D, I = self.hidden_size, self.intermediate_size
+        return [WeightSpec(self.up_name, (I, D)), WeightSpec(self.down_name, (D, I))]
+
+    def bind(self, tensors, dtype, device) -> None:
+        self.w_up, self.w_down = tensors[self.up_name], tensors[self.down_name]
+
+    def forward(self, x, residual, ctx=None) -> None:
+        if isinstance(x, LazyNorm):
+            x = x.materialize()
+        act = L.linear(x, self.w_up, None, L.STORE, glu=(PLAIN_ACTIVATIONS[self.activation], 1.0, 0.0, 0.0))
+        L.linear(act, self.w_down, None, L.RESIDUAL, residual=residual)
+
+
 register_part("ffn", "gated_mlp", GatedMLP)
+register_part("ffn", "plain_mlp", PlainMLP)

@@ -22,6 +22,9 @@ class RoutedExperts(FeedForward):
     tensor that takes part in the choice only, or none), weights = the chosen experts' scores, divided by their sum
     (+ ``renorm_eps``) with ``renormalize``, times ``route_scale``.
 
+    ``score="softmax_chosen"``: the experts with the largest logits are chosen and their weights are the softmax over the chosen
+    logits alone.  ``router_bias``: a per-expert tensor (the router's name with ``bias_ending``) joins the logits.
+
     ``groups = (count, keep)``: the router's outputs form ``count`` equal groups of neighbours, a group's score is its
     largest choice score, and only outputs of the ``keep`` best groups can be chosen.  ``identity`` = n: the router has
     ``num_experts + n`` outputs and the last n are identity experts without tensors, whose output is the input x itself
@@ -61,12 +64,13 @@ class RoutedExperts(FeedForward):
                  activation: str = "silu", names: Optional[Dict[str, str]] = None, weight_suffix: str = ".weight",
                  expert_prefix: str = "experts.", renorm_eps: float = 0.0, groups: Optional[Tuple[int, int]] = None,
                  identity: int = 0, alpha: float = 1.0, limit: Optional[float] = None, up_shift: float = 0.0,
-                 shared: Optional[Dict] = None, shared_prefix: str = "shared."):
+                 shared: Optional[Dict] = None, shared_prefix: str = "shared.", router_bias: bool = False,
+                 bias_ending: str = "bias"):
         outputs = num_experts + int(identity)
         if num_experts < 0 or identity < 0 or not 0 < top <= outputs:
             raise ValueError(f"top {top} of {num_experts} experts and {identity} identity experts")
-        if score not in ("sigmoid", "softmax"):
-            raise ValueError(f"score must be 'sigmoid' or 'softmax', got {score!r}")
+        if score not in ("sigmoid", "softmax", "softmax_chosen"):
+            raise ValueError(f"score must be 'sigmoid', 'softmax' or 'softmax_chosen', got {score!r}")
         if activation not in ("silu", "clamped_swish"):
             raise ValueError(f"routed experts implement the SiLU and the clamped swish gate, not {activation!r}")
         if activation == "clamped_swish" and (limit is None or not limit > 0):
@@ -96,6 +100,9 @@ class RoutedExperts(FeedForward):
             self.shared = {"size": int(shared["intermediate_size"]), "gate": bool(shared.get("gate", False)),
                            "glu": None if act == "silu" else (ACTIVATIONS[act], float(shared.get("alpha", alpha)),
                                                                float(shared["limit"]), float(shared.get("up_shift", up_shift)))}
+        self.has_bias = bool(router_bias)
+        self.bias_name = f"{prefix}.{self.names['router']}.{bias_ending}"
+        self.router_bias: Optional[torch.Tensor] = None
         self.w_router = self.correction = self.w_gate_up = self.w_down = self.w_down_rows = None
         self.w_shared_gate_up = self.w_shared_down = None
 
@@ -115,6 +122,8 @@ class RoutedExperts(FeedForward):
         specs = [WeightSpec(f"{self.prefix}.{self.names['router']}{self.weight_suffix}", (self.outputs, D), init=("normal", 0.1))]
         if self.has_correction:
             specs.append(WeightSpec(f"{self.prefix}.{self.names['correction']}", (self.outputs,), init=("normal", 0.1)))
+        if self.has_bias:
+            specs.append(WeightSpec(self.bias_name, (self.outputs,), init=("normal", 0.1)))
         for e in range(self.num_experts):
             specs += [WeightSpec(self._e(e, "gate"), (I, D)), WeightSpec(self._e(e, "up"), (I, D)),
                       WeightSpec(self._e(e, "down"), (D, I))]
@@ -132,6 +141,8 @@ class RoutedExperts(FeedForward):
             self.w_router = torch.cat([self.w_router, tensors[self._s("shared_gate")].float().view(1, D)]).contiguous()
         if self.has_correction:
             self.correction = tensors[f"{self.prefix}.{self.names['correction']}"].float().contiguous()
+        if self.has_bias:
+            self.router_bias = tensors[self.bias_name].float().contiguous()
         if self.shared is not None:
             g, u = tensors[self._s("gate")], tensors[self._s("up")]
             wdt = torch.float32 if torch.float32 in (g.dtype, u.dtype) else g.dtype
@@ -165,7 +176,8 @@ class RoutedExperts(FeedForward):
         gate = torch.empty((T, 1), dtype=torch.float32, device=x.device) if gated else None
         count, keep = self.groups or (0, 0)
         ops.moe_route(x, self.w_router, self.correction, self.top, self.route_scale, ids, weights, dense,
-                      softmax=self.score == "softmax", renormalize=self.renormalize, renorm_eps=self.renorm_eps,
+                      softmax="chosen" if self.score == "softmax_chosen" else self.score == "softmax",
+                      bias=self.router_bias, renormalize=self.renormalize, renorm_eps=self.renorm_eps,
                       real=self.num_experts, groups=count, keep=keep, identity_weight=idw,
                       gate_rows=1 if gated else 0, gate_out=gate)
         return ids, weights, dense, idw, gate
