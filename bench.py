@@ -5,7 +5,7 @@
     python bench.py --sizes 1.5b|7b          (the larger sizes of the family: a line of their own)
     python bench.py [--sizes ..] --only decode|prefill [--prompt-len N]     (one part, at another context length)
     python bench.py --only small-mixed       (the steps of a loaded server: a 16-token portion beside decoded tokens)
-    python bench.py --design kudadra|bulitar|kuzezen|fedirax [--sizes 1.5b] [--layers L]     (another design beside Qwen2 at equal sizes)
+    python bench.py --design kudadra|bulitar|kuzezen|fedirax|kutirax [--sizes 1.5b] [--layers L]     (another design beside Qwen2 at equal sizes)
 
 Prints one JSON line.  ``value`` is decoded tokens a second over K timed decode steps of a
 batch of 8 requests that each hold a 2,048-token prompt (random weights, random token ids),
@@ -418,6 +418,28 @@ def fedirax_config(base: dict, layers: int, kinds=("attention_2", "attention"), 
             "norm": {"eps": 1e-5}, "layers": out}
 
 
+def kutirax_config(base: dict, layers: int, kinds=("mamba2", "latent_attention"), experts: int = 8, top: int = 2,
+                   dense_first: int = 1) -> dict:
+    """A Kutirax model with the width, feed-forward, head count, head size and vocabulary of a Qwen2 configuration.  Its layers
+    cycle through ``kinds``: the state-space mixer over twice the width in heads of 64 with states of 128 in two groups and four
+    taps; latent attention with the base's heads (each of the base's head size, values alike) behind a query latent of half
+    the width and a key latent of 256, 32 rotated dimensions, a window of 1,024.  The first ``dense_first`` layers have the base's
+    dense feed-forward, the others ``experts`` experts of which ``top`` are chosen, each as wide as the dense one divided by
+    ``top``."""
+    D, H = base["hidden_size"], base["num_attention_heads"]
+    hd = base.get("head_dim", D // H)
+    mixers = {
+        "mamba2": {"heads": 2 * D // 64, "vdim": 64, "state": 128, "groups": 2, "conv": 4, "norm_groups": 2},
+        "latent_attention": {"heads": H, "dim": hd, "rot_dim": 32, "vdim": hd, "q_rank": D // 2, "kv_rank": 256,
+                             "scale": (hd + 32) ** -0.5, "rot": {"dims": 32, "base": 50000.0}, "mask": {"size": 1024}},
+    }
+    dense = {"kind": "dense", "ff": base["intermediate_size"]}
+    moe = {"kind": "moe", "expert": {"ff": base["intermediate_size"] // top}, "router": {"experts": experts, "top": top}}
+    return {"architecture": "Kutirax", "vocab": base["vocab_size"], "width": D, "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+            "layers": [{"type": kinds[i % len(kinds)], "mixer": mixers[kinds[i % len(kinds)]],
+                        "mlp": dense if i < dense_first else moe} for i in range(layers)]}
+
+
 def run_design(name: str, sizes: str, layers: int, steps: int, warmup: int, only=None) -> int:
     """Prefill of one 2,048-token prompt and decode at batch 1 / 8 / 64 over 2,048-token contexts for another design:
     its kinds of layer in turn, each kind alone, and Qwen2 with as many layer runs of the same width, feed-forward,
@@ -438,6 +460,12 @@ def run_design(name: str, sizes: str, layers: int, steps: int, warmup: int, only
                 "fedirax": fedirax_config(base, layers)}
         for kind in ("attention", "attention_2"):
             arms[f"fedirax/{kind}"] = fedirax_config(base, layers, (kind,), share=False)
+    elif name == "kutirax":
+        # beside Qwen2, Bulitar (a recurrence and attention over routed experts) and Kudadra's latent attention
+        arms = {"qwen2": base, "bulitar": bulitar_config(base, layers), "kudadra/latent_attention": kudadra_config(base, layers, ("latent_attention",)),
+                "kutirax": kutirax_config(base, layers)}
+        for kind in ("mamba2", "latent_attention"):
+            arms[f"kutirax/{kind}"] = kutirax_config(base, layers, (kind,), dense_first=layers)
     elif name == "kuzezen":
         arms = {"qwen2": base, "kuzezen": kuzezen_config(base, layers),
                 "kuzezen/no feed-forward": kuzezen_config(base, layers, ff=False)}
@@ -481,7 +509,7 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=QWEN25_05B["num_hidden_layers"])
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (for profiling runs)")
-    ap.add_argument("--design", choices=["kudadra", "bulitar", "kuzezen", "fedirax"], default=None,
+    ap.add_argument("--design", choices=["kudadra", "bulitar", "kuzezen", "fedirax", "kutirax"], default=None,
                     help="measure another design beside Qwen2 at equal sizes (0.5B sizes, or --sizes; --layers, default 6; "
                          "--only names arms, e.g. kudadra,qwen2): a line of its own, not the bench record")
     ap.add_argument("--sizes", choices=["1.5b", "7b"], default=None,

@@ -353,6 +353,83 @@ def main(argv=None) -> int:
     act_s = rn(T, I // 4, dtype=torch.bfloat16)
     run("moe_scale_one_gate_a_token", lambda: ops.moe_scale(act_s, g_gate, 1, I // 4), 2 * T * (I // 4) * 2)
 
+    # ---- token shift, attention over a rotated latent (window of 1,024), the state-space recurrence ---------------------
+    rk, rdim, qrank, window_l = 256, 32, D // 2, 1024
+    W_l = rk + rdim
+    xs_l, w1_l, mix_l, w2_l = rn(T, D), 1 + rn(D, s=0.1), rn(D, s=0.3), 1 + rn(D, s=0.1)
+    o1_l, o2_l = (torch.empty((T, D), dtype=torch.bfloat16, device=dev) for _ in range(2))
+    clear_l = torch.empty((T, D), device=dev)
+    nh, vd_s, ns, gs = 2 * D // 64, 64, 128, 2
+    chan = nh * vd_s + 2 * gs * ns
+    ssm_state = torch.zeros((max(B, 1), nh * ns * vd_s + 3 * chan + D), device=dev)
+    run("norm_shift_two_norms", lambda: ops.norm_shift(xs_l, w1_l, mix_l, 1e-5, spans1, ssm_state, nh * ns * vd_s + 3 * chan, o1_l,
+                                                       w2_l, o2_l, clear_l), T * D * (4 + 2 + 2 + 4))
+    fr_l = (1.0 / 50000.0 ** (torch.arange(0, rdim, 2, dtype=torch.float64) / rdim)).float().to(dev)
+    down_l = rn(T, qrank + W_l, dtype=torch.bfloat16)
+    cq_l = torch.empty((T, qrank), dtype=torch.bfloat16, device=dev)
+    lat_l = rn(slots, 1, W_l, dtype=torch.bfloat16)
+    nq_l, nc_l = torch.ones(qrank, device=dev), torch.ones(rk, device=dev)
+    run("latent_prepare", lambda: ops.latent_prepare(down_l, 0, qrank, qrank + rk, qrank, rk, rdim, nq_l, nc_l,
+                                                     fr_l, False, positions, positions, cq_l, lat_l, 1e-5), 2 * T * (qrank + W_l) * 2)
+    heads_l = rn(T, Hq * (hd + rdim), dtype=torch.bfloat16)
+    wk_l, wv_l = rn(Hq, rk, hd, dtype=torch.bfloat16, s=hd ** -0.5), rn(Hq, hd, rk, dtype=torch.bfloat16, s=rk ** -0.5)
+    q_l = torch.empty((T, Hq * W_l), dtype=torch.bfloat16, device=dev)
+    mixed_l = rn(T, Hq * rk, dtype=torch.bfloat16)
+    ov_l = torch.empty((T, Hq * hd), dtype=torch.bfloat16, device=dev)
+    run("head_linear_key_up_and_rotation", lambda: ops.head_linear(heads_l, 0, wk_l, q_l, x_head=hd + rdim, out_head=W_l,
+                                                                   rotate=(hd, rk, rdim, positions, fr_l, False)),
+        T * Hq * (hd + rdim + W_l) * 2, 2 * T * Hq * hd * rk)
+    run("head_linear_value_up", lambda: ops.head_linear(mixed_l, 0, wv_l, ov_l), T * Hq * (hd + rk) * 2, 2 * T * Hq * hd * rk)
+    bt_l = torch.arange(slots // page, dtype=torch.int32, device=dev).reshape(1, -1)
+    q_l = rn(T, Hq * W_l, dtype=torch.bfloat16)
+    keys_l = sum(min(p + 1, window_l) for p in range(T))
+    run("latent_attention_window_1024", lambda: ops.latent_attention(q_l, lat_l, mixed_l, z1, t1, z1, 1, bt_l, bt_l.shape[1], page, Hq,
+                                                                     W_l, rk, window_l, W_l ** -0.5, False),
+        (T * Hq * (W_l + rk) + T * W_l) * 2, 2 * Hq * (W_l + rk) * keys_l)
+    if ops.has_tcgen05() and ops.latent_attention_tcgen05_supports(W_l, rk, page):
+        run("latent_attention_tcgen05_window_1024",
+            lambda: ops.latent_attention_tcgen05(q_l, lat_l, mixed_l, z1, t1, z1, 1, bt_l, bt_l.shape[1], page, Hq, W_l, rk, window_l,
+                                                 W_l ** -0.5), (T * Hq * (W_l + rk) + T * W_l) * 2, 2 * Hq * (W_l + rk) * keys_l)
+    pages_l = -(-(C + 1) // page)
+    lat_d = rn(B * pages_l * page, 1, W_l, dtype=torch.bfloat16)
+    btd_l = torch.arange(B * pages_l, dtype=torch.int32, device=dev).reshape(B, pages_l)
+    qd_l = rn(B, Hq * W_l, dtype=torch.bfloat16)
+    od_l = torch.empty((B, Hq * rk), dtype=torch.bfloat16, device=dev)
+    for win in (window_l, 0):
+        span_l = min(C + 1, win) if win else C + 1
+        ns_l = max(1, min(ops.LATENT_MAX_SPLITS, 2 * 148 // B, span_l // 128))
+        run("latent_attention_one_token" + ("_window_1024" if win else ""),
+            lambda: ops.latent_attention(qd_l, lat_d, od_l, rB, oB, pB, B, btd_l, pages_l, page, Hq, W_l, rk, win,
+                                         W_l ** -0.5, True, ns_l), B * span_l * W_l * 2, 2 * B * Hq * (W_l + rk) * span_l)
+    in_s = rn(T, nh * vd_s + chan + nh + (-(nh * vd_s + chan + nh)) % 8, dtype=torch.bfloat16)
+    cw_s, cb_s = rn(chan, 4), rn(chan)
+    xbc_s = rn(T, chan, dtype=torch.bfloat16)
+    run("conv_act_silu", lambda: ops.conv_act(in_s, nh * vd_s, chan, cw_s, cb_s, "silu", spans1, ssm_state, nh * ns * vd_s, xbc_s),
+        2 * T * chan * 2)
+    dt_s = in_s[:, nh * vd_s + chan: nh * vd_s + chan + nh]
+    dtb_s, rate_s, skip_s = rn(nh), torch.exp(rn(nh)), rn(nh)
+    y_s = torch.empty((T, nh * vd_s), device=dev)
+    ssm = lambda n, spans, single, pieces: ops.state_space(xbc_s[:n], 0, nh * vd_s, nh * vd_s + gs * ns, dt_s[:n], dtb_s, rate_s, skip_s,
+                                                           spans, nh, gs, ns, vd_s, ssm_state, 0, y_s[:n], single, pieces)
+    ssm_bytes, ssm_flops = T * (chan * 2 + nh * vd_s * 4), 4 * T * nh * vd_s * ns
+    for piece in (128, 256, 512, 1 << 30):
+        n_p = -(-T // piece)
+        pieces_s = (i32r([0] * n_p), i32r(list(range(n_p))), i32r([0]), n_p, piece)
+        run(f"state_space_prompt_pieces_of_{piece if piece < T else T}", lambda: ssm(T, spans1, False, pieces_s), ssm_bytes, ssm_flops)
+    run("state_space_prompt_token_by_token", lambda: ssm(T, spans1, False, None), ssm_bytes, ssm_flops)
+    run("state_space_one_token", lambda: ssm(B, spansB, True, None), 2 * B * nh * ns * vd_s * 4)
+    gn_s = torch.empty((T, nh * vd_s), dtype=torch.bfloat16, device=dev)
+    gw_s = 1 + rn(nh * vd_s, s=0.1)
+    run("gated_group_norm", lambda: ops.gated_group_norm(y_s, in_s[:, :nh * vd_s], gw_s, 2, 1e-5, gn_s), T * nh * vd_s * (4 + 2 + 2))
+    if ops.has_tcgen05():
+        w_up_r, act_r = rn(I, D, dtype=torch.bfloat16, s=D ** -0.5), torch.empty((T, I), dtype=torch.bfloat16, device=dev)
+        run("up_projection_squared_relu", lambda: ops.gemm_tcgen05(x_moe, w_up_r, None, ops.EPI_STORE, act_r,
+                                                                   glu=(ops.ACT_SQUARED_RELU, 1.0, 0.0, 0.0)),
+            (T * D + I * D + T * I) * 2, 2 * T * I * D)
+    rb_s = rn(E, s=0.1)
+    run("moe_route_softmax_over_chosen", lambda: ops.moe_route(x_moe, w_router, None, top, 1.0, r_ids, r_w, r_dense, softmax="chosen",
+                                                               bias=rb_s), T * D * 2 + T * E * 4, 2 * T * D * E)
+
     # ---- what a decode step of B requests over C keys runs --------------------------------------------------------------
     pages_per = -(-(C + 1) // page)
     kcd = rn(B * pages_per * page, Hkv, hd, dtype=torch.bfloat16)

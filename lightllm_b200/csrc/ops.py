@@ -604,6 +604,29 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, sp
                                       nsplit, _f32(sinks, "sinks"), _stream()))
 
 
+def latent_attention_tcgen05_supports(width: int, rank: int, page_size: int) -> bool:
+    return bool(lib().llb_latent_attention_tcgen05_supports(width, rank, page_size))
+
+
+def latent_attention_tcgen05(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, span_row: torch.Tensor,
+                             span_len: torch.Tensor, span_pos: torch.Tensor, num_spans: int, block_table: torch.Tensor,
+                             max_pages: int, page_size: int, num_heads: int, width: int, rank: int, window: int, scale: float,
+                             sinks: Optional[torch.Tensor] = None) -> None:
+    """:func:`latent_attention` for prompt portions on the tcgen05 tensor cores (tiles of 128 (token, head) pairs)."""
+    T = q.shape[0]
+    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+        raise KernelError("latent_attention_tcgen05 takes bfloat16")
+    if q.numel() != T * num_heads * width or out.numel() != T * num_heads * rank or cache.shape[-1] != width:
+        raise KernelError("latent_attention_tcgen05: sizes do not fit")
+    if sinks is not None and sinks.numel() != num_heads:
+        raise KernelError(f"latent_attention_tcgen05: sinks must be float32 [{num_heads}]")
+    _check(lib().llb_latent_attention_tcgen05(_ptr(q), _ptr(cache), _ptr(out), T, _i32(span_row, "span_row"),
+                                              _i32(span_len, "span_len"), _i32(span_pos, "span_pos"), num_spans,
+                                              _i32(block_table, "block_table"), max_pages, page_size, cache.numel() // width,
+                                              num_heads, width, rank, window, ctypes.c_float(scale), _f32(sinks, "sinks"),
+                                              _ptr(async_error_flag(q.device)), _stream()))
+
+
 def retention(src: torch.Tensor, q_off: int, k_off: int, v_off: int, span_row: torch.Tensor, span_len: torch.Tensor,
               span_pos: torch.Tensor, span_slot: torch.Tensor, num_spans: int, num_heads: int, head_dim: int,
               v_head_dim: int, decay: torch.Tensor, inv_freq: Optional[torch.Tensor], rotary_dim: int, interleaved: bool,

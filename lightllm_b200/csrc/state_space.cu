@@ -272,13 +272,16 @@ __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint3
 
 // Shared memory of the chunk kernel.  Rows are padded by 16 bytes, so that the eight rows an ldmatrix touches lie on
 // different banks.  NP: N rounded up to 64 * MT; EV columns of x and S.
+// NST stages: with one, a block's copies wait for its work, and two blocks an SM hide each other's; with two a block alone
+// overlaps them (measured: one stage where two would leave room for a single block).
 template <int MT, int EV>
 struct ChunkShape {
+    static constexpr int NST = (MT >= 2 && EV == 64) || MT == 4 ? 1 : 2;
     static constexpr int NP = 64 * MT;
     static constexpr int NB = NP * 2 + 16;            // bytes a row of B and C
     static constexpr int XB = EV * 2 + 16;            // bytes a row of x, of its weighted halves and of S's halves
     static constexpr int STAGE = 2 * CL * NB + CL * XB;
-    static constexpr int OFF_XW = 2 * STAGE;          // weighted x: hi, lo [CL]
+    static constexpr int OFF_XW = NST * STAGE;          // weighted x: hi, lo [CL]
     static constexpr int OFF_S = OFF_XW + 2 * CL * XB;        // S before the chunk: hi, lo [NP]
     static constexpr int OFF_G = OFF_S + 2 * NP * XB;         // per stage: L [CL], dt [CL]
     static constexpr int BYTES = OFF_G + 2 * 2 * CL * 4;
@@ -287,7 +290,7 @@ struct ChunkShape {
 template <int MT, int EV, int MODE>
 __global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmParams p) {
     using Sh = ChunkShape<MT, EV>;
-    constexpr int NP = Sh::NP, NB = Sh::NB, XB = Sh::XB, NE = EV / 8, KS = NP / 16;
+    constexpr int NP = Sh::NP, NB = Sh::NB, XB = Sh::XB, NE = EV / 8, KS = NP / 16, NST = Sh::NST;
     extern __shared__ __align__(16) uint8_t smem[];
     const int item = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * EV;
     const int span = p.item_span[item], pc = p.item_c[item];
@@ -368,20 +371,21 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmParams p) {
             }
     float total = 0.0f;          // log decay over the whole piece
     const float skip = MODE == SSM_OUT ? p.skip[h] : 0.0f;
-    int stage = 0;
-    for (int c0 = 0; c0 < len; c0 += CL, stage ^= 1) {
+    int turn = 0;
+    for (int c0 = 0; c0 < len; c0 += CL, turn ^= 1) {
         const bool more = c0 + CL < len;
-        if (more) {
+        const int stage = NST == 2 ? turn : 0;
+        if (more && NST == 2) {
             fetch(c0 + CL, stage ^ 1);          // (last read before the barrier that ended the chunk before)
-            gates(c0 + CL, stage ^ 1);
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
         }
+        if (more) gates(c0 + CL, turn ^ 1);
         __syncthreads();
         const uint32_t sB = base + stage * Sh::STAGE, sC = sB + CL * NB, sX = sC + CL * NB;
         const uint8_t* gX = smem + stage * Sh::STAGE + 2 * CL * NB;
-        const float* L = reinterpret_cast<const float*>(smem + Sh::OFF_G) + stage * 2 * CL;
+        const float* L = reinterpret_cast<const float*>(smem + Sh::OFF_G) + turn * 2 * CL;
         const float* D = L + CL;
         const float Ln = L[CL - 1];
         // the weighted x of the state's update, as halves; S before the chunk, as halves
@@ -530,6 +534,7 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmParams p) {
             }
         }
         __syncthreads();          // every warp has read this stage, the weighted x and S's halves
+        if (more && NST == 1) fetch(c0 + CL, 0);
     }
     float* to = nullptr;
     if (MODE == SSM_LOCAL) {

@@ -26,8 +26,9 @@ class RotaryLatentAttentionMixer(AttentionMixer):
     the kernels see multi-query attention over the cached rows whose first ``rank`` numbers are the values, and nothing of
     the context is ever expanded.
 
-    ``window``: a query sees the latest ``window`` keys (itself included).  In bfloat16 the attention runs on the kernel of
-    csrc/latent_attention.cu, otherwise (float32, odd widths) on the CUDA-core attention kernels.  Norms, angles, scores and
+    ``window``: a query sees the latest ``window`` keys (itself included).  In bfloat16 the attention runs on the kernels of
+    csrc/latent_attention_tcgen05.cu (steps with portions of prompts) and csrc/latent_attention.cu (single tokens, latents wider
+    than 256), otherwise (float32, widths that are no multiples of 8) on the CUDA-core attention kernels.  Norms, angles, scores and
     the softmax are float32 in both precisions."""
 
     graph_safe = True
@@ -126,6 +127,11 @@ class RotaryLatentAttentionMixer(AttentionMixer):
     def attend(self, q, cache: CacheView, ctx, out) -> None:
         if not self._on_tensor_cores(q.dtype):
             super().attend(q, cache, ctx, out)
+            return
+        if not ctx.decode_only and ops.latent_attention_tcgen05_supports(self.head_dim, self.rank, ctx.page_size):
+            ops.latent_attention_tcgen05(q, cache.k, out, ctx.span_row, ctx.span_len, ctx.span_pos, ctx.num_spans,
+                                         ctx.block_tables[cache.group], ctx.max_pages, ctx.page_size, self.num_heads, self.head_dim,
+                                         self.rank, self.kernel_window(), self.scale, sinks=self.sinks)
             return
         ops.latent_attention(q, cache.k, out, ctx.span_row, ctx.span_len, ctx.span_pos, ctx.num_spans, ctx.block_tables[cache.group],
                              ctx.max_pages, ctx.page_size, self.num_heads, self.head_dim, self.rank, self.kernel_window(),
