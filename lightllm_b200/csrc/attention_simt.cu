@@ -38,6 +38,8 @@ struct AttnParams {
     const int* span_pos;
     const int* block_table;
     int max_pages, page_size, Hq, Hkv, hd, window, BQ, nsplit;
+    int share;            // groups of query heads that read one kv head of the cache: `Hkv` counts the groups, Hkv / share the cache's
+                          // heads (1 unless a group's rows would not fit in shared memory; a divisor of the heads a kv head)
     int hdv;              // width of a value row and of an output row (hd for ordinary attention)
     int vrow;             // numbers from one value row to the next (hdv; hd where values are the first hdv of the key rows)
     const float* sinks;   // [Hq] or null: exp(sinks[h]) joins the softmax denominator once, with no key and no value
@@ -58,7 +60,11 @@ __device__ __forceinline__ void store_out(const AttnParams& p, size_t i, float v
 
 // Where the value row of a slot begins for kv head kvh.
 __device__ __forceinline__ size_t value_row(const AttnParams& p, size_t slot, int kvh) {
-    return p.v_shared ? slot * (size_t)p.vrow : (slot * p.Hkv + kvh) * (size_t)p.vrow;
+    return p.v_shared ? slot * (size_t)p.vrow : (slot * (p.Hkv / p.share) + kvh / p.share) * (size_t)p.vrow;
+}
+// Where the key row of a slot begins for kv head kvh.
+__device__ __forceinline__ size_t key_row(const AttnParams& p, size_t slot, int kvh) {
+    return (slot * (p.Hkv / p.share) + kvh / p.share) * (size_t)p.hd;
 }
 
 template <typename T>
@@ -121,7 +127,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
             if (kpos < khi) {
                 const int page = bt[kpos / p.page_size];
                 const size_t slot = (size_t)page * p.page_size + (kpos % p.page_size);
-                const T* kr = kc + (slot * p.Hkv + kvh) * hd;
+                const T* kr = kc + key_row(p, slot, kvh);
                 const T* vr = vc + value_row(p, slot, kvh);
                 for (int d = lane; d < hd; d += 32) Ks[j * kstride + d] = llb_to_float(kr[d]);
                 for (int d = lane; d < hdv; d += 32) Vs[j * hdv + d] = llb_to_float(vr[d]);
@@ -316,9 +322,9 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_kernel(AttnParams p)
         for (int n = 0; n < NPMAX; ++n) acc[g][n][0] = acc[g][n][1] = 0.0f;
     }
     float* myP = Ps + warp * GMAX * 32;
-    const size_t row_stride = (size_t)p.Hkv * hd;        // of a key row
-    const size_t vrow_stride = p.v_shared ? (size_t)p.vrow : (size_t)p.Hkv * p.vrow;      // of a value row
-    const size_t vhead = p.v_shared ? 0 : (size_t)kvh * p.vrow;                    // this kv head's place in it
+    const size_t row_stride = (size_t)(p.Hkv / p.share) * hd;        // of a key row
+    const size_t vrow_stride = p.v_shared ? (size_t)p.vrow : (size_t)(p.Hkv / p.share) * p.vrow;      // of a value row
+    const size_t vhead = p.v_shared ? 0 : (size_t)(kvh / p.share) * p.vrow;        // this kv head's place in it
 
     for (int kb = klo + warp * BK; kb < khi; kb += NWARPS * BK) {
         const int kpos = kb + lane;
@@ -342,7 +348,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_kernel(AttnParams p)
 #pragma unroll
         for (int g = 0; g < GMAX; ++g) dot[g] = 0.0f;
         if (valid) {
-            const T* kr = kc + slot * row_stride + (size_t)kvh * hd;
+            const T* kr = kc + slot * row_stride + (size_t)(kvh / p.share) * hd;
 #pragma unroll 8
             for (int c = 0; c < hd; c += VEC) {
                 float kf[VEC];
@@ -505,7 +511,14 @@ size_t attention_smem_bytes(int BQ, int G, int hd, int hdv) {
 }
 
 template <typename T>
-int launch_attention(const AttnParams& p, int num_tiles, cudaStream_t stream) {
+int launch_attention(AttnParams p, int num_tiles, cudaStream_t stream) {
+    // many heads over wide rows: as many blocks share a kv head as it takes for one block's heads to fit
+    const int heads = p.Hq / p.Hkv;
+    while (p.share < heads && attention_smem_bytes(p.BQ, heads / p.share, p.hd, p.hdv) > 200 * 1024)
+        do ++p.share;
+        while (heads % p.share != 0);
+    p.Hkv *= p.share;
+    LLB_REQUIRE(p.Hkv <= 65535, "attention: too many heads");
     const size_t smem = attention_smem_bytes(p.BQ, p.Hq / p.Hkv, p.hd, p.hdv);
     LLB_REQUIRE(smem <= 220 * 1024, "attention: BQ=%d with %d heads per group and head_dim %d needs %zu bytes of "
                 "shared memory; use a smaller BQ", p.BQ, p.Hq / p.Hkv, p.hd, smem);
@@ -583,7 +596,7 @@ LLB_EXPORT int llb_paged_attention_rows(const void* q, const void* k_cache, cons
     p.max_pages = max_pages; p.page_size = page_size; p.Hq = Hq; p.Hkv = Hkv; p.hd = hd;
     p.window = window; p.BQ = BQ; p.nsplit = nsplit; p.scale = scale;
     p.softcap = softcap > 0.0f ? softcap : 0.0f;
-    p.hdv = hdv; p.vrow = vrow; p.sinks = sinks;
+    p.hdv = hdv; p.vrow = vrow; p.sinks = sinks; p.share = 1;
     LLB_REQUIRE(vrow >= hdv, "attention: value rows of %d numbers, %d apart", hdv, vrow);
     p.v_shared = v_shared ? 1 : 0; p.out_f32 = out_f32 ? 1 : 0;
     p.part_acc = scratch;

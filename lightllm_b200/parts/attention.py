@@ -15,7 +15,6 @@ from .base import CacheView, LazyNorm, Mixer, Part
 
 # Shared memory budget per block used to pick the tile height of the CUDA-core kernel.
 _SMEM_BUDGET = 100 * 1024
-_SMEM_LIMIT = 200 * 1024
 # Portions of at least this many rows run on the tensor-core attention kernel (tiles of 128 rows, the rows beyond the
 # portion masked): one block of the CUDA-core kernel walking a portion's keys takes hundreds of microseconds from a
 # few hundred keys on, an item of the tensor-core kernel about two per 128 keys.
@@ -220,14 +219,13 @@ class AttentionMixer(Mixer):
         return q
 
     def tile_height(self) -> int:
+        """Query rows a tile of the CUDA-core kernel: as many as the shared memory holds (one row always runs: the kernel
+        shares a kv head's query heads among blocks when even one row of all of them does not fit)."""
         group = self.num_heads // self.num_kv_heads
-        for bq in (16, 8, 4, 2, 1):
-            need = ops.attention_smem_bytes(bq, group, self.head_dim, self.v_head_dim * self.value_cross)
-            if need <= _SMEM_BUDGET or (bq == 1 and need <= _SMEM_LIMIT):
+        for bq in (16, 8, 4, 2):
+            if ops.attention_smem_bytes(bq, group, self.head_dim, self.v_head_dim * self.value_cross) <= _SMEM_BUDGET:
                 return bq
-        raise ops.KernelError(
-            f"attention with {group} query heads per kv head and head_dim {self.head_dim} does not fit "
-            f"in shared memory even with one query row per block")
+        return 1
 
     def _plan(self, ctx, dtype):
         """Which kernels this step's attention takes and over which tiles: made once per step (in
