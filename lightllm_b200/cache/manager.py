@@ -115,7 +115,7 @@ class SeqCache:
     slot: int
     length: int = 0
     tables: List[List[int]] = field(default_factory=list)
-    first_live: List[int] = field(default_factory=list)    # first logical page not yet released
+    first_live: List[int] = field(default_factory=list)    # first logical page that no window has passed yet
     version: int = 0                                       # bumped whenever a table changes
     _np: Dict[int, Any] = field(default_factory=dict)      # group -> (version, int32 array of the table)
 
@@ -243,7 +243,8 @@ class CacheManager:
                 first_needed_pos = max(first_needed_pos, new_len - new_len % spec.chunk)
             dead = max(0, first_needed_pos) // self.page_size   # logical pages wholly before it
             table = seq.tables[g]
-            for lp in range(seq.first_live[g], min(dead, len(table))):
+            kept = -(-spec.keep_first // self.page_size)           # logical pages of the first positions, which stay visible
+            for lp in range(max(seq.first_live[g], kept), min(dead, len(table))):
                 self.pools[g].give(table[lp], seq_id)
                 table[lp] = -1
                 seq.version += 1

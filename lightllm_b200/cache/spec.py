@@ -17,13 +17,16 @@ class KVSpec:
     ``window`` = how many of the latest positions (the token itself included) stay visible; ``None`` = all of
     them.  ``v_head_dim``: ``None`` = as wide as the keys; 0 = no values are kept (a mixer that reads its values
     out of the key rows, e.g. attention over a shared latent).  ``chunk``: a query only sees the positions of its own
-    block of ``chunk`` positions (blocks counted from position 0), so the pages of earlier blocks are given back."""
+    block of ``chunk`` positions (blocks counted from position 0), so the pages of earlier blocks are given back.
+    ``keep_first``: beside a window's latest positions the first ``keep_first`` of the sequence stay visible, so their pages
+    are held until the request ends."""
 
     kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_head_dim: Optional[int] = None
     chunk: Optional[int] = None
+    keep_first: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -82,6 +85,9 @@ class CacheLayout:
                 if want is not None and have.window is not None and (want.window is None or want.window > have.window):
                     raise ValueError(
                         f"run entry {i} needs a window of {want.window} but entry {src} keeps only {have.window} keys")
+                if want is not None and have.window is not None and want.keep_first > have.keep_first:
+                    raise ValueError(
+                        f"run entry {i} needs the first {want.keep_first} positions but entry {src} keeps {have.keep_first}")
                 ref = PlaneRef(owner.group, owner.plane, owner.state_plane, owns=False)
             elif spec is not None:
                 if spec.kv is not None:

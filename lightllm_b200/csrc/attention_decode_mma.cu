@@ -40,6 +40,8 @@ struct DecodeParams {
     int max_pages, page_size, Hq, Hkv, window, nsplit;
     float scale_log2e;
     float cap_log2e, inv_cap;      // a soft cap on the scores: cap * log2(e) and scale / cap (0: no cap)
+    int keep;                      // the first `keep` positions stay visible whatever the window says
+    const float* slopes;           // [Hq] or null: slopes[h] * (query position - key position) is taken off the (capped) score
     float* part_acc;               // [tiles, Hkv, nsplit, G, HD]
     float* part_ml;                // [tiles, Hkv, nsplit, G, 2]   (m in base-2 units, l)
     const float* sinks;            // [Hq] or null: exp(sinks[h]) joins head h's softmax denominator once
@@ -108,21 +110,21 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_mma_kernel(DecodePar
     const int row0 = p.span_row[span] + q0;
     const int qpos = p.span_pos[span] + q0;
     const int* bt = p.block_table + (size_t)span * p.max_pages;
-    const int hi = qpos + 1;
-    const int lo = llb_first_visible(qpos, p.window);
-    int klo = lo, khi = hi;
+    // the visible keys, numbered without the gap between the kept first positions and the window
+    const LlbKeys keys = llb_keys(llb_first_visible(qpos, p.window), qpos + 1, p.keep);
+    int klo = 0, khi = keys.count;
     if (p.nsplit > 1) {
-        int chunk = (hi - lo + p.nsplit - 1) / p.nsplit;
+        int chunk = (keys.count + p.nsplit - 1) / p.nsplit;
         chunk = ((chunk + BK - 1) / BK) * BK;
-        klo = lo + split * chunk;
-        khi = min(hi, klo + chunk);
+        klo = split * chunk;
+        khi = min(keys.count, klo + chunk);
     }
     const size_t row_stride = (size_t)p.Hkv * HD;
     // cache row of this lane's key in a tile that starts at kb (only block tables are read: no dependency)
     // (an int: a row of a head is 128 bytes or more, so a plane of 2^31 rows would not fit the device's memory)
     auto slot_of = [&](int kb) -> int {
-        const int kpos = kb + lane;
-        if (lane >= BK || kpos >= khi) return -1;
+        if (lane >= BK || kb + lane >= khi) return -1;
+        const int kpos = keys.pos(kb + lane);
         return bt[kpos / p.page_size] * p.page_size + (kpos % p.page_size);
     };
     const int kb_first = klo + warp * BK;
@@ -170,6 +172,12 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_mma_kernel(DecodePar
 #pragma unroll
     for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
+    float slope[2] = {0.0f, 0.0f};          // of this lane's two rows, in base-2 units
+    if (p.slopes) {
+        const int r0 = lane >> 2;
+        if (r0 < G) slope[0] = p.slopes[kvh * G + r0] * 1.4426950408889634f;
+        if (r0 + 8 < G) slope[1] = p.slopes[kvh * G + r0 + 8] * 1.4426950408889634f;
+    }
 
     int buf = 0;
 #pragma unroll
@@ -215,6 +223,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_mma_kernel(DecodePar
                     } else {
                         v = s[i][e] * p.scale_log2e;
                     }
+                    if (p.slopes) v -= slope[e >> 1] * (float)(qpos - keys.pos(key));
                 }
                 s[i][e] = v;
                 mt[e >> 1] = fmaxf(mt[e >> 1], v);
@@ -515,12 +524,14 @@ LLB_EXPORT int llb_paged_decode_mma_cluster_splits() { return CLUSTER_MAX_SPLITS
 // cross > 1 (then = Hkv, and no sinks): crossed values, out is [T, Hq, cross, hd] and holds every query head's
 // weights applied to the values of every kv head; scratch counts Hq * cross heads.  out_float: out is float, not bf16.
 // softcap > 0: every score (after `scale`) becomes softcap * tanh(score / softcap) before the softmax; sinks are not capped.
-LLB_EXPORT int llb_paged_decode_mma_capped(const void* q, const void* k_cache, const void* v_cache, void* out,
+// keep: the first `keep` positions stay visible whatever the window says (0: none).  slopes [Hq] float or null: slopes[h] *
+// (query position - key position) is taken off head h's scores after the cap; sinks carry no such bias.
+LLB_EXPORT int llb_paged_decode_mma_biased(const void* q, const void* k_cache, const void* v_cache, void* out,
                                            const int* tile_span, const int* tile_q0, int num_tiles, const int* span_row,
                                            const int* span_pos, const int* block_table, int max_pages, int page_size,
                                            int Hq, int Hkv, int hd, int window, float scale, float softcap, int nsplit,
                                            float* scratch, const float* sinks, int cross, int out_float,
-                                           cudaStream_t stream) {
+                                           int keep, const float* slopes, cudaStream_t stream) {
     if (num_tiles == 0) return 0;
     LLB_REQUIRE(cross == 1 || (cross == Hkv && sinks == nullptr),
                 "decode attention: crossed values take cross = the number of kv heads (%d), got %d, and no sinks", Hkv, cross);
@@ -538,6 +549,9 @@ LLB_EXPORT int llb_paged_decode_mma_capped(const void* q, const void* k_cache, c
     p.window = window; p.nsplit = nsplit; p.scale_log2e = scale * 1.4426950408889634f;
     p.cap_log2e = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
     p.inv_cap = softcap > 0.0f ? scale / softcap : 0.0f;
+    LLB_REQUIRE(keep >= 0, "decode attention: %d kept first positions", keep);
+    p.keep = keep;
+    p.slopes = slopes;
     p.sinks = sinks;
     p.cross = cross;
     p.out_f32 = out_float ? (float*)out : nullptr;
@@ -546,6 +560,17 @@ LLB_EXPORT int llb_paged_decode_mma_capped(const void* q, const void* k_cache, c
     p.part_ml = scratch ? scratch + (size_t)num_tiles * Hkv * cross * nsplit * G * hd : nullptr;
     if (hd == 64) return launch<64>(p, num_tiles, stream);
     return launch<128>(p, num_tiles, stream);
+}
+
+LLB_EXPORT int llb_paged_decode_mma_capped(const void* q, const void* k_cache, const void* v_cache, void* out,
+                                           const int* tile_span, const int* tile_q0, int num_tiles, const int* span_row,
+                                           const int* span_pos, const int* block_table, int max_pages, int page_size,
+                                           int Hq, int Hkv, int hd, int window, float scale, float softcap, int nsplit,
+                                           float* scratch, const float* sinks, int cross, int out_float,
+                                           cudaStream_t stream) {
+    return llb_paged_decode_mma_biased(q, k_cache, v_cache, out, tile_span, tile_q0, num_tiles, span_row, span_pos,
+        block_table, max_pages, page_size, Hq, Hkv, hd, window, scale, softcap, nsplit, scratch, sinks, cross,
+        out_float, 0, nullptr, stream);
 }
 
 LLB_EXPORT int llb_paged_decode_mma_cross(const void* q, const void* k_cache, const void* v_cache, void* out,

@@ -47,6 +47,8 @@ struct AttnParams {
     int out_f32;          // out is float whatever the dtype of q and the caches
     float scale;
     float softcap;        // > 0: a score s becomes softcap * tanh(s / softcap) before the softmax; 0: scores as they are
+    int keep;             // the first `keep` positions stay visible whatever the window says
+    const float* slopes;  // [Hq] or null: slopes[h] * (query position - key position) is taken off the (capped) score
     float* part_acc;  // [tiles, Hkv, nsplit, BQ*G, hdv]
     float* part_ml;   // [tiles, Hkv, nsplit, BQ*G, 2]
 };
@@ -95,15 +97,15 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
     const T* kc = (const T*)p.k_cache;
     const T* vc = (const T*)p.v_cache;
 
-    // Key range of the tile: [lo, hi); of this split: [klo, khi).
-    const int hi = pos0 + nrows;
-    const int lo = llb_first_visible(pos0, p.window);
-    int klo = lo, khi = hi;
+    // The keys of the tile, numbered without the gap between the kept first positions and the window; of this split:
+    // numbers [klo, khi).
+    const LlbKeys keys = llb_keys(llb_first_visible(pos0, p.window), pos0 + nrows, p.keep);
+    int klo = 0, khi = keys.count;
     if (p.nsplit > 1) {
-        int chunk = (hi - lo + p.nsplit - 1) / p.nsplit;
+        int chunk = (keys.count + p.nsplit - 1) / p.nsplit;
         chunk = ((chunk + BK - 1) / BK) * BK;
-        klo = lo + split * chunk;
-        khi = min(hi, klo + chunk);
+        klo = split * chunk;
+        khi = min(keys.count, klo + chunk);
     }
 
     for (int i = threadIdx.x; i < nqv * hd; i += blockDim.x) {
@@ -123,8 +125,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
     for (int kb = klo; kb < khi; kb += BK) {
         // Stage BK keys and values of this kv head; rows past khi are zero.
         for (int j = warp; j < BK; j += NWARPS) {
-            const int kpos = kb + j;
-            if (kpos < khi) {
+            if (kb + j < khi) {
+                const int kpos = keys.pos(kb + j);
                 const int page = bt[kpos / p.page_size];
                 const size_t slot = (size_t)page * p.page_size + (kpos % p.page_size);
                 const T* kr = kc + key_row(p, slot, kvh);
@@ -138,12 +140,12 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
         }
         __syncthreads();
 
-        const int kpos = kb + lane;
+        const int kpos = keys.pos(kb + lane);
         for (int v = warp; v < nqv; v += NWARPS) {
             const int r = v / G;
             if (r >= nrows) continue;  // uniform over the warp
             const int qpos = pos0 + r;
-            const bool visible = kpos < khi && kpos <= qpos && kpos >= llb_first_visible(qpos, p.window);
+            const bool visible = kb + lane < khi && kpos <= qpos && (kpos >= llb_first_visible(qpos, p.window) || kpos < p.keep);
             float s = -INFINITY;
             if (visible) {
                 const float* qv = Qs + (size_t)v * hd;
@@ -152,6 +154,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_kernel(AttnParams
                 for (int d = 0; d < hd; ++d) dot = fmaf(qv[d], kr[d], dot);
                 s = dot * p.scale;
                 if (p.softcap > 0.0f) s = p.softcap * tanhf(s / p.softcap);
+                if (p.slopes) s -= p.slopes[kvh * G + (v - r * G)] * (float)(qpos - kpos);
             }
             const float m_old = Ms[v];
             const float m_new = fmaxf(m_old, llb_warp_max(s));
@@ -300,14 +303,13 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_kernel(AttnParams p)
     const T* kc = (const T*)p.k_cache;
     const T* vc = (const T*)p.v_cache;
 
-    const int hi = qpos + 1;
-    const int lo = llb_first_visible(qpos, p.window);
-    int klo = lo, khi = hi;
+    const LlbKeys keys = llb_keys(llb_first_visible(qpos, p.window), qpos + 1, p.keep);
+    int klo = 0, khi = keys.count;
     if (p.nsplit > 1) {
-        int chunk = (hi - lo + p.nsplit - 1) / p.nsplit;
+        int chunk = (keys.count + p.nsplit - 1) / p.nsplit;
         chunk = ((chunk + BK - 1) / BK) * BK;
-        klo = lo + split * chunk;
-        khi = min(hi, klo + chunk);
+        klo = split * chunk;
+        khi = min(keys.count, klo + chunk);
     }
     for (int i = threadIdx.x; i < G * hd; i += blockDim.x)
         Qs[i] = llb_to_float(q[((size_t)row0 * p.Hq + kvh * G) * hd + i]);
@@ -327,8 +329,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_kernel(AttnParams p)
     const size_t vhead = p.v_shared ? 0 : (size_t)(kvh / p.share) * p.vrow;        // this kv head's place in it
 
     for (int kb = klo + warp * BK; kb < khi; kb += NWARPS * BK) {
-        const int kpos = kb + lane;
-        const bool valid = kpos < khi;
+        const int kpos = keys.pos(kb + lane);
+        const bool valid = kb + lane < khi;
         const int nkeys = min(BK, khi - kb);
         size_t slot = 0;
         if (valid) slot = (size_t)bt[kpos / p.page_size] * p.page_size + (kpos % p.page_size);
@@ -370,6 +372,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_decode_kernel(AttnParams p)
                 if (valid) {
                     sc = dot[g] * p.scale;
                     if (p.softcap > 0.0f) sc = p.softcap * tanhf(sc / p.softcap);
+                    if (p.slopes) sc -= p.slopes[kvh * G + g] * (float)(qpos - kpos);
                 }
                 const float m_new = fmaxf(m[g], llb_warp_max(sc));      // finite: the tile has a valid key
                 const float pr = valid ? expf(sc - m_new) : 0.0f;
@@ -576,12 +579,14 @@ LLB_EXPORT long long llb_attention_scratch_floats(int num_tiles, int Hq, int hd,
 // softcap > 0: every score (after `scale`) becomes softcap * tanh(score / softcap); sinks are not capped.
 // vrow: numbers from one (slot, kv head)'s value row to the next; hdv, or hd with v_cache == k_cache: the values are the first
 // hdv numbers of the key rows.
-LLB_EXPORT int llb_paged_attention_rows(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
+// keep: the first `keep` positions stay visible whatever the window says (0: none).  slopes [Hq] float or null: slopes[h] *
+// (query position - key position) is taken off head h's scores after the cap; sinks carry no such bias.
+LLB_EXPORT int llb_paged_attention_biased(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
                                         const int* tile_span, const int* tile_q0, int num_tiles, const int* span_row,
                                         const int* span_len, const int* span_pos, const int* block_table,
                                         int max_pages, int page_size, int Hq, int Hkv, int hd, int hdv, int vrow,
                                         const float* sinks, int window, float scale, float softcap, int BQ, int nsplit,
-                                        float* scratch, int v_shared, int out_f32, cudaStream_t stream) {
+                                        float* scratch, int v_shared, int out_f32, int keep, const float* slopes, cudaStream_t stream) {
     if (num_tiles == 0) return 0;
     LLB_REQUIRE(num_tiles > 0 && Hq > 0 && Hkv > 0 && hd > 0 && hdv > 0 && page_size > 0 && max_pages > 0 && BQ > 0,
                 "attention: bad sizes");
@@ -598,12 +603,26 @@ LLB_EXPORT int llb_paged_attention_rows(const void* q, const void* k_cache, cons
     p.softcap = softcap > 0.0f ? softcap : 0.0f;
     p.hdv = hdv; p.vrow = vrow; p.sinks = sinks; p.share = 1;
     LLB_REQUIRE(vrow >= hdv, "attention: value rows of %d numbers, %d apart", hdv, vrow);
+    LLB_REQUIRE(keep >= 0, "attention: %d kept first positions", keep);
+    p.keep = keep; p.slopes = slopes;
     p.v_shared = v_shared ? 1 : 0; p.out_f32 = out_f32 ? 1 : 0;
     p.part_acc = scratch;
     p.part_ml = scratch ? scratch + (size_t)num_tiles * Hq * BQ * nsplit * hdv : nullptr;
     if (dtype == LLB_F32) return launch_attention<float>(p, num_tiles, stream);
     if (dtype == LLB_BF16) return launch_attention<__nv_bfloat16>(p, num_tiles, stream);
     return llb_fail("attention: unknown dtype %d", dtype);
+}
+
+LLB_EXPORT int llb_paged_attention_rows(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
+                                        const int* tile_span, const int* tile_q0, int num_tiles, const int* span_row,
+                                        const int* span_len, const int* span_pos, const int* block_table,
+                                        int max_pages, int page_size, int Hq, int Hkv, int hd, int hdv, int vrow,
+                                        const float* sinks, int window, float scale, float softcap, int BQ, int nsplit,
+                                        float* scratch, int v_shared, int out_f32, cudaStream_t stream) {
+    return llb_paged_attention_biased(q, k_cache, v_cache, out, dtype, tile_span, tile_q0, num_tiles, span_row,
+                                      span_len, span_pos, block_table, max_pages, page_size, Hq, Hkv, hd, hdv, vrow,
+                                      sinks, window, scale, softcap, BQ, nsplit, scratch, v_shared, out_f32, 0,
+                                      nullptr, stream);
 }
 
 LLB_EXPORT int llb_paged_attention_capped(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,

@@ -39,13 +39,17 @@ constexpr int NUM_THREADS = 320;   // 8 softmax warps (two threads per query row
 constexpr int MMA_WARP = 8, LOAD_WARP = 9;
 
 // Masking is a select on the column index, never a branch: columns c_lo .. c_hi of the tile are this row's
-// visible keys (causal, the span's end, the window's start; c_hi < c_lo when none is).
-__device__ __forceinline__ float masked(float s, int col, int c_lo, int c_hi) {
-    return (col >= c_lo && col <= c_hi) ? s : -INFINITY;
+// visible keys (causal, the span's end, the window's start; c_hi < c_lo when none is), and of the columns before c_keep
+// (kept first positions) those up to c_hi.
+struct Visible {
+    int lo, hi, keep;
+};
+__device__ __forceinline__ float masked(float s, int col, const Visible& c) {
+    return ((col >= c.lo || col < c.keep) && col <= c.hi) ? s : -INFINITY;
 }
 // Largest raw score of this thread's row among the visible keys of its two 32-column chunks of the tile.
 template <bool MASKED>
-__device__ __forceinline__ float row_max(uint32_t tmem_s, int c_begin, int c_lo, int c_hi) {
+__device__ __forceinline__ float row_max(uint32_t tmem_s, int c_begin, const Visible& vis) {
     float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
 #pragma unroll 1
     for (int c = c_begin; c < c_begin + 2; ++c) {
@@ -53,7 +57,7 @@ __device__ __forceinline__ float row_max(uint32_t tmem_s, int c_begin, int c_lo,
         tmem_ld32(tmem_s + c * 32, s);
         if (MASKED) {
 #pragma unroll
-            for (int i = 0; i < 32; ++i) s[i] = masked(s[i], c * 32 + i, c_lo, c_hi);
+            for (int i = 0; i < 32; ++i) s[i] = masked(s[i], c * 32 + i, vis);
         }
 #pragma unroll
         for (int i = 0; i < 32; i += 4) {
@@ -70,12 +74,45 @@ __device__ __forceinline__ float capped_score(float s, float inv_cap, float cap_
     const float t = 1.0f - __fdividef(2.0f, 1.0f + fast_exp2(x * 2.8853900817779268f));
     return s == -INFINITY ? -INFINITY : t * cap_log2e;
 }
+// A bias by distance: slope * (query position - key position) is taken off the score.  Everything in base-2 units; `at`
+// is slope times the query's column in the tile, so that column c has the bias slope * c - at.
+struct Bias {
+    float slope, at;
+};
+// With a bias the largest raw score need not give the largest score, and scoring every key twice would double the tile's
+// exponentials under a cap.  What the softmax wants is a shift that no score exceeds by much or falls short of by much:
+// the largest raw score of 8 neighbouring keys, capped, with the bias of their last one.  It is at most 7 slopes above the
+// true maximum of the 8 (a masked key's column can only raise it, by as little).
+template <bool MASKED, bool CAPPED>
+__device__ __forceinline__ float row_bound(uint32_t tmem_s, int c_begin, float c_scale, float cap_log2e, const Bias& b, const Visible& vis) {
+    float m0 = -INFINITY, m1 = -INFINITY;
+#pragma unroll 1
+    for (int c = c_begin; c < c_begin + 2; ++c) {
+        float s[32];
+        tmem_ld32(tmem_s + c * 32, s);
+        if (MASKED) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) s[i] = masked(s[i], c * 32 + i, vis);
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            float g = fmaxf(fmaxf(fmaxf(s[8 * q], s[8 * q + 1]), fmaxf(s[8 * q + 2], s[8 * q + 3])),
+                            fmaxf(fmaxf(s[8 * q + 4], s[8 * q + 5]), fmaxf(s[8 * q + 6], s[8 * q + 7])));
+            g = CAPPED ? capped_score(g, c_scale, cap_log2e) : g * c_scale;
+            g += fmaf(b.slope, (float)(c * 32 + 8 * q + 7), -b.at);
+            if (q & 1) m1 = fmaxf(m1, g);
+            else m0 = fmaxf(m0, g);
+        }
+    }
+    return fmaxf(m0, m1);
+}
 // p = 2^(s*c - m) of this thread's 64 scores of the row, written as bf16 into the swizzled A-operand tiles; returns
 // their sum (float, before rounding).  Row r, 16-byte chunk q of a 128-byte row lands at chunk q ^ (r & 7).
-// CAPPED: c_scale is scale / cap and the score in base-2 units is capped_score(s, c_scale, cap_log2e).
-template <bool MASKED, bool CAPPED = false>
+// CAPPED: c_scale is scale / cap and the score in base-2 units is capped_score(s, c_scale, cap_log2e).  BIASED: with the
+// bias `b`.
+template <bool MASKED, bool CAPPED, bool BIASED>
 __device__ __forceinline__ float row_probs(uint32_t tmem_s, uint8_t* p_s, int r, int c_begin, float c_scale, float m_use,
-                                           int c_lo, int c_hi, float cap_log2e = 0.0f) {
+                                           const Visible& vis, float cap_log2e, const Bias& b) {
     float l0 = 0.0f, l1 = 0.0f;
 #pragma unroll 1
     for (int c = c_begin; c < c_begin + 2; ++c) {
@@ -83,21 +120,27 @@ __device__ __forceinline__ float row_probs(uint32_t tmem_s, uint8_t* p_s, int r,
         tmem_ld32(tmem_s + c * 32, s);
         if (MASKED) {
 #pragma unroll
-            for (int i = 0; i < 32; ++i) s[i] = masked(s[i], c * 32 + i, c_lo, c_hi);
+            for (int i = 0; i < 32; ++i) s[i] = masked(s[i], c * 32 + i, vis);
         }
         uint8_t* prow = p_s + (c >> 1) * (128 * 128) + (uint32_t)r * 128;
+        // what a score is shifted by: -m, and with a bias the one of the chunk's first column
+        const float shift = BIASED ? fmaf(b.slope, (float)(c * 32), -b.at) - m_use : -m_use;
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
             uint32_t w[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                float p0, p1;
+                float p0, p1, t0 = shift, t1 = shift;
+                if (BIASED) {
+                    t0 = fmaf(b.slope, (float)(q * 8 + 2 * e), shift);
+                    t1 = fmaf(b.slope, (float)(q * 8 + 2 * e + 1), shift);
+                }
                 if (CAPPED) {
-                    p0 = fast_exp2(capped_score(s[q * 8 + 2 * e], c_scale, cap_log2e) - m_use);
-                    p1 = fast_exp2(capped_score(s[q * 8 + 2 * e + 1], c_scale, cap_log2e) - m_use);
+                    p0 = fast_exp2(capped_score(s[q * 8 + 2 * e], c_scale, cap_log2e) + t0);
+                    p1 = fast_exp2(capped_score(s[q * 8 + 2 * e + 1], c_scale, cap_log2e) + t1);
                 } else {
-                    p0 = fast_exp2(fmaf(s[q * 8 + 2 * e], c_scale, -m_use));
-                    p1 = fast_exp2(fmaf(s[q * 8 + 2 * e + 1], c_scale, -m_use));
+                    p0 = fast_exp2(fmaf(s[q * 8 + 2 * e], c_scale, t0));
+                    p1 = fast_exp2(fmaf(s[q * 8 + 2 * e + 1], c_scale, t1));
                 }
                 l0 += p0;
                 l1 += p1;
@@ -122,6 +165,8 @@ struct AttnTcParams {
     int max_pages, page_size, Hq, Hkv, window, num_slots, num_items;
     float scale_log2e;         // scale * log2(e): scores are kept in base-2 units
     float cap_log2e, inv_cap;  // a soft cap on the scores: cap * log2(e) and scale / cap (0: no cap), see capped_score
+    int keep;                  // the first `keep` positions stay visible whatever the window says
+    const float* slopes;       // [Hq] or null: slopes[h] * (query position - key position) is taken off the (capped) score
     uint32_t dynamic_smem_bytes;
     // Optional cut of a tile's key range into work items, so that long rows do not set the kernel's time:
     // item i covers key tiles [tile_k0[i], tile_k0[i] + tile_nk[i]) of its query tile and, when tile_part[i] >= 0,
@@ -142,8 +187,15 @@ struct AttnTcParams {
 
 // What one work item is: 128 query rows of one span and one head over a range of key tiles.
 struct Item {
-    int head, span, row0, nrows, pos0, hi, lo, kt0, ntiles, part;
+    int head, span, row0, nrows, pos0, hi, lo, ntiles, part;
     int qhead;      // the query head; `head` is where the result goes (the same unless values are crossed)
+    // The key tiles of a row tile: those of the kept first positions that lie before the window's first tile, then the
+    // window's.  Tile j of the item is number first + j of them.
+    int first, head_tiles, gap;      // gap: what is added to a window tile's number to give its place among all tiles of 128 keys
+    __device__ __forceinline__ int key(int j) const {
+        const int n = first + j;
+        return (n < head_tiles ? n : n + gap) * BKV;
+    }
 };
 __device__ __forceinline__ Item make_item(const AttnTcParams& p, int idx) {
     Item it;
@@ -157,9 +209,11 @@ __device__ __forceinline__ Item make_item(const AttnTcParams& p, int idx) {
     it.pos0 = p.span_pos[it.span] + q0;
     it.hi = it.pos0 + it.nrows;                                    // keys [lo, hi) can be visible
     it.lo = llb_first_visible(it.pos0, p.window);
-    const int k_first = p.tile_k0 ? p.tile_k0[tile] : 0;
-    it.kt0 = (it.lo / BKV) * BKV + k_first * BKV;
-    const int all_tiles = (it.hi - (it.lo / BKV) * BKV + BKV - 1) / BKV - k_first;
+    it.first = p.tile_k0 ? p.tile_k0[tile] : 0;
+    const int lo_tile = it.lo / BKV;
+    it.head_tiles = min((p.keep + BKV - 1) / BKV, lo_tile);
+    it.gap = lo_tile - it.head_tiles;
+    const int all_tiles = it.head_tiles + (it.hi - lo_tile * BKV + BKV - 1) / BKV - it.first;
     it.ntiles = max(0, p.tile_nk ? min(p.tile_nk[tile], all_tiles) : all_tiles);
     it.part = p.tile_part ? p.tile_part[tile] : -1;
     return it;
@@ -181,9 +235,9 @@ __device__ __forceinline__ void named_barrier(int id, int threads) {
 // The roles meet on mbarriers (data arrived, buffers free, tensor-core work done; every wait is bounded) and on
 // named barriers among softmax and MMA warps.  After a wait has run out every role still walks through all its
 // items and barriers, without copies, tensor-core work or stores, so that no barrier is left waiting.
-// CAP: the scores carry a soft cap (p.cap_log2e, p.inv_cap); a kernel of its own, so that the plain one keeps its
-// registers.
-template <int HD, bool CAP>
+// CAP: the scores carry a soft cap (p.cap_log2e, p.inv_cap); BIAS: a bias by distance (p.slopes).  Kernels of their own, so
+// that the plain one keeps its registers.
+template <int HD, bool CAP, bool BIAS>
 __global__ void __launch_bounds__(NUM_THREADS, HD <= 64 ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const AttnTcParams p) {
@@ -271,12 +325,12 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             }
             for (int j = 0; j < it.ntiles; ++j, ++n_kv) {
                 const int st = n_kv & 1;
-                const int kt = it.kt0 + j * BKV;
+                const int kt = it.key(j);
                 // page numbers first: their latency then lies under the wait for the stage
                 const int ppt = BKV / p.page_size;
                 const int lp = kt / p.page_size + lane;
-                // only pages that hold keys of [lo, hi): what lies beyond the request's own keys is never read
-                const bool holds_keys = lp * p.page_size < it.hi && (lp + 1) * p.page_size > it.lo;
+                // only pages that hold keys of [lo, hi) or kept ones: what lies beyond the request's own keys is never read
+                const bool holds_keys = lp * p.page_size < it.hi && ((lp + 1) * p.page_size > it.lo || lp * p.page_size < p.keep);
                 const int page = (lane < ppt && lp < p.max_pages && holds_keys) ? bt[lp] : -1;
                 if (n_kv >= 2) ok = mbar_wait(&bar_kv_free[st], ((n_kv >> 1) - 1) & 1, abort_flag) && ok;
                 if (!ok) continue;
@@ -377,8 +431,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
             for (int d = 0; d < HO; ++d) o[d] = 0.0f;
             float m_run = -INFINITY, l_run = 0.0f;
+            const float slope = BIAS ? p.slopes[it.qhead] * 1.4426950408889634f : 0.0f;
             for (int j = 0; j < it.ntiles; ++j, ++n_s) {
-                const int kt = it.kt0 + j * BKV;
+                const int kt = it.key(j);
                 if (j == 0) {      // later tiles' S came with the commit behind the tile before them
                     ok = mbar_wait(bar_s, n_item & 1, abort_flag) && ok;
                     if (threadIdx.x == 0 && it.ntiles == 1) mbar_arrive(bar_q_free);     // the item's last S has read Q
@@ -399,25 +454,29 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 // Softmax of this thread's row over its 64 keys of the tile, in two passes over tensor memory
                 // (maximum first, then the probabilities), 32 columns at a time.  Tiles that lie wholly below
                 // the diagonal and inside the window of every row of the block skip the masking.
-                const bool interior = (kt + BKV - 1 <= it.pos0) && kt >= llb_first_visible(it.pos0 + BQ - 1, p.window);
-                const int c_lo = vis_lo - kt, c_hi = vis_hi - kt;
+                const bool interior = (kt + BKV - 1 <= it.pos0) &&
+                                      (kt >= llb_first_visible(it.pos0 + BQ - 1, p.window) || kt + BKV <= p.keep);
+                const Visible vis = {vis_lo - kt, vis_hi - kt, p.keep - kt};
+                const Bias bias = {slope, slope * (float)(qpos - kt)};
+                const float c_scale = CAP ? p.inv_cap : p.scale_log2e;
                 float m_tile;
-                if (interior) m_tile = row_max<false>(tmem_s, 2 * half, c_lo, c_hi);
-                else m_tile = row_max<true>(tmem_s, 2 * half, c_lo, c_hi);
+                if (BIAS) {
+                    if (interior) m_tile = row_bound<false, CAP>(tmem_s, 2 * half, c_scale, p.cap_log2e, bias, vis);
+                    else m_tile = row_bound<true, CAP>(tmem_s, 2 * half, c_scale, p.cap_log2e, bias, vis);
+                } else if (interior) m_tile = row_max<false>(tmem_s, 2 * half, vis);
+                else m_tile = row_max<true>(tmem_s, 2 * half, vis);
                 xch[half][r] = __float2bfloat16_ru(m_tile);      // rewritten only after the barriers further down
                 named_barrier(BAR_SOFTMAX, NUM_SOFTMAX);
                 m_tile = fmaxf(__bfloat162float(xch[0][r]), __bfloat162float(xch[1][r]));
                 // the scale is positive and the cap grows with the score: the largest raw score gives the largest capped one
-                m_tile = CAP ? capped_score(m_tile, p.inv_cap, p.cap_log2e) : m_tile * p.scale_log2e;
+                // (a bound with a bias is in base-2 units already)
+                if (!BIAS) m_tile = CAP ? capped_score(m_tile, p.inv_cap, p.cap_log2e) : m_tile * p.scale_log2e;
                 const float m_new = fmaxf(m_run, m_tile);
                 const float m_use = (m_new == -INFINITY) ? 0.0f : m_new;      // nothing visible yet: all p are 0
                 const float corr = (m_run == -INFINITY) ? 0.0f : fast_exp2(m_run - m_use);
                 float l_tile;
-                if (CAP) {
-                    if (interior) l_tile = row_probs<false, true>(tmem_s, p_s, r, 2 * half, p.inv_cap, m_use, c_lo, c_hi, p.cap_log2e);
-                    else l_tile = row_probs<true, true>(tmem_s, p_s, r, 2 * half, p.inv_cap, m_use, c_lo, c_hi, p.cap_log2e);
-                } else if (interior) l_tile = row_probs<false>(tmem_s, p_s, r, 2 * half, p.scale_log2e, m_use, c_lo, c_hi);
-                else l_tile = row_probs<true>(tmem_s, p_s, r, 2 * half, p.scale_log2e, m_use, c_lo, c_hi);
+                if (interior) l_tile = row_probs<false, CAP, BIAS>(tmem_s, p_s, r, 2 * half, c_scale, m_use, vis, p.cap_log2e, bias);
+                else l_tile = row_probs<true, CAP, BIAS>(tmem_s, p_s, r, 2 * half, c_scale, m_use, vis, p.cap_log2e, bias);
                 l_run = l_run * corr + l_tile;
                 m_run = m_new;
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");       // P is read by the tensor core
@@ -559,7 +618,7 @@ int make_map(const void* ptr, long long rows, long long cols, int box_rows, CUte
     return make_map_bf16(ptr, rows, cols, box_rows, out);
 }
 
-template <int HD, bool CAP>
+template <int HD, bool CAP, bool BIAS>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcParams& p, int num_tiles,
            cudaStream_t stream) {
     constexpr int KB = HD / 64;
@@ -568,7 +627,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     constexpr size_t smem = (size_t)(KB + 4 * KB + 2) * 128 * 128 + 1024 - 592;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<HD, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<HD, CAP, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              (int)smem);
         if (e != cudaSuccess) return llb_fail("attention_tcgen05: cannot opt in to %zu bytes of shared memory: %s", smem,
                                               cudaGetErrorString(e));
@@ -598,7 +657,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    cudaError_t e = cudaLaunchKernelEx(&cfg, attention_tcgen05_kernel<HD, CAP>, mq, mk, mv, pp);
+    cudaError_t e = cudaLaunchKernelEx(&cfg, attention_tcgen05_kernel<HD, CAP, BIAS>, mq, mk, mv, pp);
     if (e != cudaSuccess) return llb_fail("attention_tcgen05: launch failed: %s", cudaGetErrorString(e));
     return llb_check_launch("attention_tcgen05");
 }
@@ -620,14 +679,17 @@ LLB_EXPORT int llb_attention_tcgen05_supports(int hd, int page_size) {
 // cross > 1 (then = Hkv, and no sinks): crossed values.  out is float [T, Hq, cross, hd] and holds every query head's
 // weights applied to the values of every kv head; part_scratch and the merge count Hq * cross heads.
 // softcap > 0: every score (after `scale`) becomes softcap * tanh(score / softcap) before the softmax; sinks are not capped.
-LLB_EXPORT int llb_paged_attention_tcgen05_capped(const void* q, const void* k_cache, const void* v_cache, void* out, int T,
+// keep: the first `keep` positions stay visible whatever the window says (0: none); the tiles of a row tile are then those of
+// the kept positions before the window's first tile, followed by the window's, and tile_k0 / tile_nk count them so.  slopes [Hq]
+// float or null: slopes[h] * (query position - key position) is taken off head h's scores after the cap; sinks carry no bias.
+LLB_EXPORT int llb_paged_attention_tcgen05_biased(const void* q, const void* k_cache, const void* v_cache, void* out, int T,
                                                   const int* tile_span, const int* tile_q0, int num_tiles,
                                                   const int* span_row, const int* span_len, const int* span_pos,
                                                   const int* block_table, int max_pages, int page_size, int num_slots,
                                                   int Hq, int Hkv, int hd, int window, float scale, float softcap,
                                                   const int* tile_k0, const int* tile_nk, const int* tile_part,
                                                   float* part_scratch, int num_parts, const float* sinks, int cross,
-                                                  int out_float, int* error_flag, cudaStream_t stream) {
+                                                  int out_float, int* error_flag, int keep, const float* slopes, cudaStream_t stream) {
     if (num_tiles == 0) return 0;
     LLB_REQUIRE(cross == 1 || (cross == Hkv && sinks == nullptr),
                 "attention_tcgen05: crossed values take cross = the number of kv heads (%d), got %d, and no sinks", Hkv, cross);
@@ -654,13 +716,32 @@ LLB_EXPORT int llb_paged_attention_tcgen05_capped(const void* q, const void* k_c
     p.cap_log2e = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
     p.inv_cap = softcap > 0.0f ? scale / softcap : 0.0f;
     p.tile_k0 = tile_k0; p.tile_nk = tile_nk; p.tile_part = tile_part;
+    LLB_REQUIRE(keep >= 0, "attention_tcgen05: %d kept first positions", keep);
+    p.keep = keep; p.slopes = slopes;
     p.sinks = sinks;
     p.part_o = part_scratch;
     p.part_ml = part_scratch ? part_scratch + (size_t)num_parts * Hq * cross * BQ * hd : nullptr;
-    if (p.cap_log2e > 0.0f)
-        return hd == 64 ? launch<64, true>(mq, mk, mv, p, num_tiles, stream) : launch<128, true>(mq, mk, mv, p, num_tiles, stream);
-    if (hd == 64) return launch<64, false>(mq, mk, mv, p, num_tiles, stream);
-    return launch<128, false>(mq, mk, mv, p, num_tiles, stream);
+    const bool cap = p.cap_log2e > 0.0f, bias = slopes != nullptr;
+    if (hd == 64) {
+        if (bias) return cap ? launch<64, true, true>(mq, mk, mv, p, num_tiles, stream) : launch<64, false, true>(mq, mk, mv, p, num_tiles, stream);
+        return cap ? launch<64, true, false>(mq, mk, mv, p, num_tiles, stream) : launch<64, false, false>(mq, mk, mv, p, num_tiles, stream);
+    }
+    if (bias) return cap ? launch<128, true, true>(mq, mk, mv, p, num_tiles, stream) : launch<128, false, true>(mq, mk, mv, p, num_tiles, stream);
+    return cap ? launch<128, true, false>(mq, mk, mv, p, num_tiles, stream) : launch<128, false, false>(mq, mk, mv, p, num_tiles, stream);
+}
+
+LLB_EXPORT int llb_paged_attention_tcgen05_capped(const void* q, const void* k_cache, const void* v_cache, void* out, int T,
+                                                  const int* tile_span, const int* tile_q0, int num_tiles,
+                                                  const int* span_row, const int* span_len, const int* span_pos,
+                                                  const int* block_table, int max_pages, int page_size, int num_slots,
+                                                  int Hq, int Hkv, int hd, int window, float scale, float softcap,
+                                                  const int* tile_k0, const int* tile_nk, const int* tile_part,
+                                                  float* part_scratch, int num_parts, const float* sinks, int cross,
+                                                  int out_float, int* error_flag, cudaStream_t stream) {
+    return llb_paged_attention_tcgen05_biased(q, k_cache, v_cache, out, T, tile_span, tile_q0, num_tiles, span_row,
+        span_len, span_pos, block_table, max_pages, page_size, num_slots, Hq, Hkv, hd, window, scale, softcap,
+        tile_k0, tile_nk, tile_part, part_scratch, num_parts, sinks, cross, out_float, error_flag, 0, nullptr,
+        stream);
 }
 
 LLB_EXPORT int llb_paged_attention_tcgen05_cross(const void* q, const void* k_cache, const void* v_cache, void* out, int T,

@@ -77,11 +77,14 @@ struct LlbGluArgs {
 // The store epilogue of a contraction takes the same arguments with the kinds of a plain activation (no gate):
 //   LLB_ACT_SQUARED_RELU   max(v, 0)^2          anything else: v
 enum LlbAct { LLB_ACT_SQUARED_RELU = 16 };
+// ... and the float store and residual epilogues the kind LLB_OUT_SCALE: every output (bias included) times `alpha`.
+enum LlbOut { LLB_OUT_SCALE = 17 };
 __device__ __forceinline__ float llb_act(float v, int kind) {
     if (kind != LLB_ACT_SQUARED_RELU) return v;
     v = fmaxf(v, 0.0f);
     return v * v;
 }
+__device__ __forceinline__ float llb_out_scale(const LlbGluArgs& g) { return g.kind == LLB_OUT_SCALE ? g.alpha : 1.0f; }
 static inline LlbGluArgs llb_glu_silu() { return LlbGluArgs{LLB_GLU_SILU, 1.0f, 0.0f, 0.0f}; }
 
 static inline int llb_ceil_div(int a, int b) { return (a + b - 1) / b; }
@@ -96,4 +99,20 @@ __host__ __device__ __forceinline__ int llb_first_visible(int qpos, int window) 
     if (window > 0) return qpos - window + 1 > 0 ? qpos - window + 1 : 0;
     if (window < 0) return qpos - qpos % (-window);
     return 0;
+}
+
+// The keys of a query whose first `keep` positions stay visible besides those from `lo` (= llb_first_visible) to `hi` - 1:
+// the kept positions that lie before lo and then lo .. hi - 1, numbered one after the other without the gap between them.
+struct LlbKeys {
+    int kept;      // how many of the numbers are kept positions before lo
+    int gap;       // what is added to every later number to give its position
+    int count;     // numbers in all
+    __host__ __device__ __forceinline__ int pos(int v) const { return v < kept ? v : v + gap; }
+};
+__host__ __device__ __forceinline__ LlbKeys llb_keys(int lo, int hi, int keep) {
+    LlbKeys k;
+    k.kept = keep < lo ? keep : lo;
+    k.gap = lo - k.kept;
+    k.count = hi - k.gap;
+    return k;
 }

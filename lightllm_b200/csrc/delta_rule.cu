@@ -1,6 +1,10 @@
-// The gated delta rule with one decay per head and key channel, as a recurrence over a per-request state in float:
+// The gated delta rule with one decay per head and key channel (or one per head), as a recurrence over a per-request state in
+// float:
 //
 //     S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t          S [dim, vdim] per head
+//
+// One decay a head: g_t is a number, exp(-rate_h * softplus(a_t + dt_bias_h)), made inside the kernels from a column a head of
+// a fused projection (template flag HEAD).
 //
 // in this order, so the read-out sees the token's own write.  The state is zero before a request's first token and lives
 // in the request's state slot between steps, so any cutting of the tokens gives the same recurrence.
@@ -29,7 +33,10 @@ struct DeltaParams {
     const float* q;            // [T, G, dim]
     const float* k;            // [T, G, dim]
     const float* v;            // [T, H, vdim]
-    const float* g;            // [T, H, dim] logarithms of the decay factors (<= 0)
+    const float* g;            // [T, H, dim] logarithms of the decay factors (<= 0); null: one decay a head, from
+    const void* a;             //   row t at a + t * beta_stride elements (beta_dtype): H values,
+    const float* dt_bias;      //   [H],
+    const float* rate;         //   [H]: the logarithm is -rate_h * softplus(a_h + dt_bias_h)
     const void* beta;          // row t at beta + t * beta_stride elements: H values before the sigmoid
     long long beta_stride;
     int beta_dtype;
@@ -47,7 +54,17 @@ struct DeltaParams {
     int nr, dg;                // blocked: the second kernel's split of a column (rows a thread, threads a column)
 };
 
-template <int NR, int DG>
+// The value before the sigmoid (beta) or the softplus (a) of head h in row `row`.
+__device__ __forceinline__ float delta_gate_in(const DeltaParams& p, const void* base, size_t row, int h) {
+    const size_t at = row * (size_t)p.beta_stride + h;
+    return p.beta_dtype == LLB_F32 ? ((const float*)base)[at] : __bfloat162float(((const __nv_bfloat16*)base)[at]);
+}
+__device__ __forceinline__ float delta_head_log_decay(const DeltaParams& p, size_t row, int h) {
+    const float z = delta_gate_in(p, p.a, row, h) + p.dt_bias[h];
+    return -p.rate[h] * (z > 20.0f ? z : log1pf(expf(z)));
+}
+
+template <int NR, int DG, bool HEAD>
 __global__ void __launch_bounds__(256) delta_rule_kernel(DeltaParams p) {
     extern __shared__ __align__(16) float sm[];
     constexpr int PADF = delta_pad(NR, DG);
@@ -58,8 +75,9 @@ __global__ void __launch_bounds__(256) delta_rule_kernel(DeltaParams p) {
     float* qs = sm;                              // [STAGE][DPAD]
     float* ks = qs + DELTA_STAGE * DPAD;
     float* gs = ks + DELTA_STAGE * DPAD;
-    float* vs = gs + DELTA_STAGE * DPAD;         // [STAGE][EV]
+    float* vs = HEAD ? gs : gs + DELTA_STAGE * DPAD;         // [STAGE][EV]  (one decay a head: no rows of decays)
     float* bs = vs + DELTA_STAGE * p.EV;         // [STAGE]
+    float* hs = bs + DELTA_STAGE;                // [STAGE] the head's decays
     const int dg = threadIdx.x % DG, el = threadIdx.x / DG;
     const int e = blockIdx.z * p.EV + el;
     const bool live = el < p.EV && e < vdim;
@@ -72,7 +90,7 @@ __global__ void __launch_bounds__(256) delta_rule_kernel(DeltaParams p) {
         const int d = dg * NR + j;
         S[j] = (pos0 > 0 && live && d < dim) ? slot[(size_t)d * vdim + e] : 0.0f;
     }
-    for (int i = threadIdx.x; i < 3 * DELTA_STAGE * DPAD; i += blockDim.x) sm[i] = 0.0f;     // the padding stays zero
+    for (int i = threadIdx.x; i < (HEAD ? 2 : 3) * DELTA_STAGE * DPAD; i += blockDim.x) sm[i] = 0.0f;     // the padding stays zero
     auto at = [](int d) { return (d / NR) * (NR + PADF) + d % NR; };
     for (int c0 = 0; c0 < len; c0 += DELTA_STAGE) {
         const int n = min(DELTA_STAGE, len - c0);
@@ -82,7 +100,7 @@ __global__ void __launch_bounds__(256) delta_rule_kernel(DeltaParams p) {
             const size_t row = (size_t)(row0 + c0 + tl);
             qs[tl * DPAD + at(d)] = p.q[(row * p.G + hk) * dim + d];
             ks[tl * DPAD + at(d)] = p.k[(row * p.G + hk) * dim + d];
-            gs[tl * DPAD + at(d)] = expf(p.g[(row * p.H + h) * dim + d]);
+            if (!HEAD) gs[tl * DPAD + at(d)] = expf(p.g[(row * p.H + h) * dim + d]);
         }
         for (int it = threadIdx.x; it < n * p.EV; it += blockDim.x) {
             const int tl = it / p.EV, cc = it - tl * p.EV;
@@ -90,15 +108,14 @@ __global__ void __launch_bounds__(256) delta_rule_kernel(DeltaParams p) {
             vs[it] = ee < vdim ? p.v[((size_t)(row0 + c0 + tl) * p.H + h) * vdim + ee] : 0.0f;
         }
         if (threadIdx.x < n) {
-            const size_t at_b = (size_t)(row0 + c0 + threadIdx.x) * p.beta_stride + h;
-            const float z = p.beta_dtype == LLB_F32 ? ((const float*)p.beta)[at_b]
-                                                    : __bfloat162float(((const __nv_bfloat16*)p.beta)[at_b]);
-            bs[threadIdx.x] = 1.0f / (1.0f + expf(-z));
+            bs[threadIdx.x] = 1.0f / (1.0f + expf(-delta_gate_in(p, p.beta, (size_t)(row0 + c0 + threadIdx.x), h)));
+            if (HEAD) hs[threadIdx.x] = expf(delta_head_log_decay(p, (size_t)(row0 + c0 + threadIdx.x), h));
         }
         __syncthreads();
         for (int tl = 0; tl < n; ++tl) {
             const float vv = el < p.EV ? vs[tl * p.EV + el] : 0.0f;
             const float beta = bs[tl];
+            const float gh = HEAD ? hs[tl] : 1.0f;
             const float4* k4p = reinterpret_cast<const float4*>(ks + tl * DPAD + dg * (NR + PADF));
             const float4* q4p = reinterpret_cast<const float4*>(qs + tl * DPAD + dg * (NR + PADF));
             const float4* g4p = reinterpret_cast<const float4*>(gs + tl * DPAD + dg * (NR + PADF));
@@ -106,7 +123,7 @@ __global__ void __launch_bounds__(256) delta_rule_kernel(DeltaParams p) {
             float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
 #pragma unroll
             for (int j = 0; j < NR; j += 4) {
-                const float4 g4 = g4p[j >> 2];
+                const float4 g4 = HEAD ? make_float4(gh, gh, gh, gh) : g4p[j >> 2];
                 const float4 k4 = kk[j >> 2] = k4p[j >> 2];
                 S[j] *= g4.x; S[j + 1] *= g4.y; S[j + 2] *= g4.z; S[j + 3] *= g4.w;
                 a0 = fmaf(S[j], k4.x, a0); a1 = fmaf(S[j + 1], k4.y, a1);
@@ -163,11 +180,14 @@ __host__ __device__ inline long long delta_block_floats(int dpad) {
     return 3ll * DELTA_STAGE * dpad + dpad + 2 * DELTA_STAGE * DELTA_STAGE;
 }
 
+template <bool HEAD>
 __global__ void __launch_bounds__(256) delta_blocks_prepare_kernel(DeltaParams p, int num_spans) {
     extern __shared__ __align__(16) float sm[];
     constexpr int C = DELTA_STAGE;
     const int dim = p.dim, h = blockIdx.y;
     const int RS = dim + 1;                      // row pitch: the rows of a warp's pairs on different banks
+    const int LS = HEAD ? 1 : RS;                // pitch of the log decays
+    const int decays = HEAD ? 1 : dim;           // of a token
     int span = 0, c = blockIdx.x;
     while (span < num_spans) {
         const int blocks = (p.span_len[span] + C - 1) / C;
@@ -181,7 +201,7 @@ __global__ void __launch_bounds__(256) delta_blocks_prepare_kernel(DeltaParams p
     const int hk = h / (p.H / p.G);
     float* kr = sm;                              // [C][RS]    k_t
     float* qr = kr + C * RS;                     // [C][RS]    q_t
-    float* Ls = qr + C * RS;                     // [C][RS]    log decays, then their running sums L_t
+    float* Ls = qr + C * RS;                     // [C][LS]    log decays, then their running sums L_t
     const int nr = p.nr, padded = p.nr + delta_pad(p.nr, p.dg), dpad = p.dg * padded;
     float* dst = p.scratch + ((size_t)blockIdx.x * p.H + h) * delta_block_floats(dpad);
     float* Qb = dst;                             // [C][dpad]  e^{L_t} q_t
@@ -196,20 +216,22 @@ __global__ void __launch_bounds__(256) delta_blocks_prepare_kernel(DeltaParams p
         const bool in = tl < n;
         kr[tl * RS + d] = in ? p.k[(row * p.G + hk) * dim + d] : 0.0f;
         qr[tl * RS + d] = in ? p.q[(row * p.G + hk) * dim + d] : 0.0f;
-        Ls[tl * RS + d] = in ? p.g[(row * p.H + h) * dim + d] : 0.0f;
+        if (!HEAD) Ls[tl * LS + d] = in ? p.g[(row * p.H + h) * dim + d] : 0.0f;
     }
+    if (HEAD && threadIdx.x < C) Ls[threadIdx.x] = threadIdx.x < n ? delta_head_log_decay(p, (size_t)(row0 + threadIdx.x), h) : 0.0f;
     __syncthreads();
-    for (int d = threadIdx.x; d < dim; d += blockDim.x) {          // running sums of the log decays
+    for (int d = threadIdx.x; d < decays; d += blockDim.x) {          // running sums of the log decays
         float run = 0.0f;
         for (int tl = 0; tl < C; ++tl) {
-            run += Ls[tl * RS + d];
-            Ls[tl * RS + d] = run;
+            run += Ls[tl * LS + d];
+            Ls[tl * LS + d] = run;
         }
     }
     __syncthreads();
     for (int it = threadIdx.x; it < C * dim; it += blockDim.x) {
         const int tl = it / dim, d = it - tl * dim;
-        const float L = Ls[tl * RS + d], Ln = Ls[(C - 1) * RS + d];          // rows past n add nothing: L stays L_n
+        const int ld = HEAD ? 0 : d;
+        const float L = Ls[tl * LS + ld], Ln = Ls[(C - 1) * LS + ld];          // rows past n add nothing: L stays L_n
         const float eL = expf(L);
         const int col = (d / nr) * padded + d % nr;
         Kb[tl * dpad + col] = eL * kr[tl * RS + d];
@@ -236,9 +258,14 @@ __global__ void __launch_bounds__(256) delta_blocks_prepare_kernel(DeltaParams p
         float a = 0.0f, m = 0.0f;
         if (t < n) {
             for (int d = 0; d < dim; ++d) {
-                const float w = kr[s * RS + d] * expf(Ls[t * RS + d] - Ls[s * RS + d]);
+                const float w = HEAD ? kr[s * RS + d] : kr[s * RS + d] * expf(Ls[t * LS + d] - Ls[s * LS + d]);
                 a = fmaf(kr[t * RS + d], w, a);
                 m = fmaf(qr[t * RS + d], w, m);
+            }
+            if (HEAD) {
+                const float e = expf(Ls[t] - Ls[s]);
+                a *= e;
+                m *= e;
             }
         }
         As[s * C + t] = s < t ? a : 0.0f;
@@ -291,10 +318,7 @@ __global__ void __launch_bounds__(64) delta_rule_blocked_kernel(DeltaParams p) {
             vnext[i] = (it < C * p.EV && tl < n && ee < vdim) ? p.v[((size_t)(row0 + c0 + tl) * p.H + h) * vdim + ee] : 0.0f;
         }
         bnext = -INFINITY;          // (its sigmoid is 0; taken when the value is stored, not while the load is in flight)
-        if (threadIdx.x < n) {
-            const size_t at_b = (size_t)(row0 + c0 + threadIdx.x) * p.beta_stride + h;
-            bnext = p.beta_dtype == LLB_F32 ? ((const float*)p.beta)[at_b] : __bfloat162float(((const __nv_bfloat16*)p.beta)[at_b]);
-        }
+        if (threadIdx.x < n) bnext = delta_gate_in(p, p.beta, (size_t)(row0 + c0 + threadIdx.x), h);
     };
     auto store_vb = [&](int stage) {
         float* vsn = sm + stage * stage_pitch + BLOCK_FLOATS;
@@ -408,13 +432,13 @@ __global__ void __launch_bounds__(64) delta_rule_blocked_kernel(DeltaParams p) {
     }
 }
 
-template <int NR, int DG>
-int launch_delta(const DeltaParams& p0, int num_spans, cudaStream_t stream) {
+template <int NR, int DG, bool HEAD>
+int launch_delta_as(const DeltaParams& p0, int num_spans, cudaStream_t stream) {
     DeltaParams p = p0;
     const int cols = 256 / DG;
     p.EV = p.vdim < cols ? p.vdim : cols;
     constexpr int PADF = delta_pad(NR, DG);
-    const size_t smem = (size_t)(3 * DELTA_STAGE * DG * (NR + PADF) + DELTA_STAGE * p.EV + DELTA_STAGE) * sizeof(float);
+    const size_t smem = (size_t)((HEAD ? 2 : 3) * DELTA_STAGE * DG * (NR + PADF) + DELTA_STAGE * p.EV + 2 * DELTA_STAGE) * sizeof(float);
     const int threads = ((p.EV * DG + 31) / 32) * 32;
     const dim3 grid(num_spans, p.H, (p.vdim + p.EV - 1) / p.EV);
     if (p.blocked) {
@@ -427,12 +451,12 @@ int launch_delta(const DeltaParams& p0, int num_spans, cudaStream_t stream) {
         const dim3 grid_b(num_spans, p.H, (p.vdim + p.EV - 1) / p.EV);
         const size_t pre_bytes = (size_t)3 * C * (p.dim + 1) * sizeof(float);
         if (pre_bytes > 48 * 1024) {
-            const cudaError_t e = cudaFuncSetAttribute(delta_blocks_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+            const cudaError_t e = cudaFuncSetAttribute(delta_blocks_prepare_kernel<HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                        (int)pre_bytes);
             if (e != cudaSuccess) return llb_fail("delta_rule: %s", cudaGetErrorString(e));
         }
         p.nr = NR; p.dg = DG;
-        delta_blocks_prepare_kernel<<<dim3(p.max_blocks, p.H), 256, pre_bytes, stream>>>(p, num_spans);
+        delta_blocks_prepare_kernel<HEAD><<<dim3(p.max_blocks, p.H), 256, pre_bytes, stream>>>(p, num_spans);
         int rc = llb_check_launch("delta_blocks_prepare");
         if (rc) return rc;
         const size_t stage = ((size_t)delta_block_floats(DG * (NR + PADF)) + C * p.EV + C + 3) & ~(size_t)3;
@@ -446,11 +470,16 @@ int launch_delta(const DeltaParams& p0, int num_spans, cudaStream_t stream) {
         return llb_check_launch("delta_rule_blocked");
     }
     if (smem > 48 * 1024) {
-        const cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<NR, DG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<NR, DG, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return llb_fail("delta_rule: %s", cudaGetErrorString(e));
     }
-    delta_rule_kernel<NR, DG><<<grid, threads, smem, stream>>>(p);
+    delta_rule_kernel<NR, DG, HEAD><<<grid, threads, smem, stream>>>(p);
     return llb_check_launch("delta_rule");
+}
+
+template <int NR, int DG>
+int launch_delta(const DeltaParams& p, int num_spans, cudaStream_t stream) {
+    return p.g ? launch_delta_as<NR, DG, false>(p, num_spans, stream) : launch_delta_as<NR, DG, true>(p, num_spans, stream);
 }
 
 struct LowRankParams {
@@ -462,7 +491,13 @@ struct LowRankParams {
     const float* rate;         // [N / per_rate] (mode 2)
     void* out;                 // [T, N]
     int mode;
+    float inv_tau;             // (mode 3)
 };
+
+// ln(sigmoid(z)) = -softplus(-z), from the side that loses nothing.
+__device__ __forceinline__ float llb_log_sigmoid(float z) {
+    return z < 0.0f ? z - log1pf(expf(z)) : -log1pf(expf(-z));
+}
 
 // A block takes LR_ROWS rows of x (their R inputs in shared memory, padded to a multiple of 4) and 256 outputs; a thread
 // owns one output for all the block's rows, so a weight is loaded once for LR_ROWS products and the inputs come as
@@ -511,6 +546,8 @@ __global__ void __launch_bounds__(256) low_rank_up_kernel(LowRankParams p, int T
         } else if (p.mode == 2) {
             const float sp = z > 20.0f ? z : log1pf(expf(z));
             z = -rate * sp;
+        } else if (p.mode == 3) {
+            z = p.inv_tau * llb_log_sigmoid(z);
         }
         ((TO*)p.out)[(size_t)(t0 + tl) * p.N + n] = llb_from_float<TO>(z);
     }
@@ -520,6 +557,7 @@ __device__ __forceinline__ float low_rank_finish(const LowRankParams& p, int n, 
     if (p.bias) z += p.bias[n];
     if (p.mode == 1) return 1.0f / (1.0f + expf(-z));
     if (p.mode == 2) return -p.rate[n / p.per_rate] * (z > 20.0f ? z : log1pf(expf(z)));
+    if (p.mode == 3) return p.inv_tau * llb_log_sigmoid(z);
     return z;
 }
 
@@ -568,25 +606,20 @@ int launch_low_rank(const LowRankParams& p, int T, int out_dtype, cudaStream_t s
 
 }  // namespace
 
-// q, k float [T, G, dim]; v float [T, H, vdim]; g float [T, H, dim] (the logarithms of the decay factors, <= 0); blocked != 0
-// walks the spans in blocks of tokens (for steps with long spans; the result is the same recurrence) and needs scratch of
-// llb_delta_rule_scratch_floats(max_blocks, H, dim) floats, max_blocks >= sum over spans of ceil(len / 16) (T / 16 +
-// num_spans always suffices); beta: the H values
-// before the sigmoid of row t at beta + t * beta_stride (float or bf16); the spans of the step; state: float base of the
-// state plane, state_stride floats a slot, a slot's S [H, dim, vdim] at state_off; out float [T, H, vdim].
-LLB_EXPORT int llb_delta_rule(const float* q, const float* k, const float* v, const float* g, const void* beta,
+static int delta_rule_impl(const float* q, const float* k, const float* v, const float* g, const void* a, const float* dt_bias,
+                           const float* rate, const void* beta,
                               long long beta_stride, int beta_dtype, const int* span_row, const int* span_len,
                               const int* span_pos, const int* span_slot, int num_spans, int H, int G, int dim, int vdim,
                               float* state, long long state_stride, long long state_off, float* out, int blocked,
                               float* scratch, int max_blocks, cudaStream_t stream) {
     if (num_spans == 0) return 0;
-    LLB_REQUIRE(q && k && v && g && beta && state && out && span_row && span_len && span_pos && span_slot,
+    LLB_REQUIRE(q && k && v && (g || (a && dt_bias && rate)) && beta && state && out && span_row && span_len && span_pos && span_slot,
                 "delta_rule: bad arguments");
     LLB_REQUIRE(H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0, "delta_rule: bad sizes H=%d G=%d dim=%d vdim=%d", H, G, dim, vdim);
     LLB_REQUIRE(dim <= 256, "delta_rule: heads of %d key channels; at most 256", dim);
     LLB_REQUIRE(beta_dtype == LLB_F32 || beta_dtype == LLB_BF16, "delta_rule: unknown dtype %d", beta_dtype);
     DeltaParams p;
-    p.q = q; p.k = k; p.v = v; p.g = g; p.beta = beta; p.beta_stride = beta_stride; p.beta_dtype = beta_dtype;
+    p.q = q; p.k = k; p.v = v; p.g = g; p.a = a; p.dt_bias = dt_bias; p.rate = rate; p.beta = beta; p.beta_stride = beta_stride; p.beta_dtype = beta_dtype;
     p.span_row = span_row; p.span_len = span_len; p.span_pos = span_pos; p.span_slot = span_slot;
     p.state = state; p.state_stride = state_stride; p.state_off = state_off; p.out = out;
     p.H = H; p.G = G; p.dim = dim; p.vdim = vdim; p.EV = 0; p.blocked = blocked;
@@ -606,6 +639,35 @@ LLB_EXPORT int llb_delta_rule(const float* q, const float* k, const float* v, co
     return launch_delta<32, 8>(p, num_spans, stream);
 }
 
+// q, k float [T, G, dim]; v float [T, H, vdim]; g float [T, H, dim] (the logarithms of the decay factors, <= 0); blocked != 0
+// walks the spans in blocks of tokens (for steps with long spans; the result is the same recurrence) and needs scratch of
+// llb_delta_rule_scratch_floats(max_blocks, H, dim) floats, max_blocks >= sum over spans of ceil(len / 16) (T / 16 +
+// num_spans always suffices); beta: the H values
+// before the sigmoid of row t at beta + t * beta_stride (float or bf16); the spans of the step; state: float base of the
+// state plane, state_stride floats a slot, a slot's S [H, dim, vdim] at state_off; out float [T, H, vdim].
+LLB_EXPORT int llb_delta_rule(const float* q, const float* k, const float* v, const float* g, const void* beta,
+                              long long beta_stride, int beta_dtype, const int* span_row, const int* span_len,
+                              const int* span_pos, const int* span_slot, int num_spans, int H, int G, int dim, int vdim,
+                              float* state, long long state_stride, long long state_off, float* out, int blocked,
+                              float* scratch, int max_blocks, cudaStream_t stream) {
+    return delta_rule_impl(q, k, v, g, nullptr, nullptr, nullptr, beta, beta_stride, beta_dtype, span_row, span_len,
+        span_pos, span_slot, num_spans, H, G, dim, vdim, state, state_stride, state_off, out, blocked, scratch,
+        max_blocks, stream);
+}
+
+// The same with one decay a head: its logarithm is -rate[h] * softplus(a[t, h] + dt_bias[h]); row t of `a` begins at
+// a + t * beta_stride elements and has beta's dtype (columns of the same fused projection); dt_bias, rate float [H].
+LLB_EXPORT int llb_delta_rule_head(const float* q, const float* k, const float* v, const void* a, const float* dt_bias,
+                                   const float* rate, const void* beta,
+                              long long beta_stride, int beta_dtype, const int* span_row, const int* span_len,
+                              const int* span_pos, const int* span_slot, int num_spans, int H, int G, int dim, int vdim,
+                              float* state, long long state_stride, long long state_off, float* out, int blocked,
+                              float* scratch, int max_blocks, cudaStream_t stream) {
+    return delta_rule_impl(q, k, v, nullptr, a, dt_bias, rate, beta, beta_stride, beta_dtype, span_row, span_len,
+        span_pos, span_slot, num_spans, H, G, dim, vdim, state, state_stride, state_off, out, blocked, scratch,
+        max_blocks, stream);
+}
+
 LLB_EXPORT long long llb_delta_rule_scratch_floats(int max_blocks, int H, int dim) {
     const int nr = dim <= 64 ? 4 : dim <= 128 ? 8 : 16;          // as llb_delta_rule picks them
     const int dg = dim <= 16 ? 4 : dim <= 32 ? 8 : 16;
@@ -614,21 +676,29 @@ LLB_EXPORT long long llb_delta_rule_scratch_floats(int max_blocks, int H, int di
 
 // out[t, n] = f(sum_r x[t, x_off + r] * w[n, r] + bias[n]) for T rows of x (row stride x_stride elements, float or bf16),
 // w [N, R] float or bf16, bias float [N] or null, out [T, N] float or bf16.  mode 0: f = identity; 1: sigmoid;
-// 2: -rate[n / per_rate] * softplus(.), the logarithm of a decay factor, rate float [N / per_rate].
-LLB_EXPORT int llb_low_rank_up(const void* x, int x_dtype, long long x_stride, int x_off, int T, int R, const void* w,
+// 2: -rate[n / per_rate] * softplus(.), the logarithm of a decay factor, rate float [N / per_rate]; 3 (llb_low_rank_up_tau):
+// inv_tau * ln(sigmoid(.)), the logarithm of sigmoid(.)^(1 / tau).
+LLB_EXPORT int llb_low_rank_up_tau(const void* x, int x_dtype, long long x_stride, int x_off, int T, int R, const void* w,
                                int w_dtype, int N, const float* bias, int mode, const float* rate, int per_rate,
-                               void* out, int out_dtype, cudaStream_t stream) {
+                               float inv_tau, void* out, int out_dtype, cudaStream_t stream) {
     if (T == 0 || N == 0) return 0;
     LLB_REQUIRE(T > 0 && R > 0 && N > 0 && x && w && out, "low_rank_up: bad arguments");
-    LLB_REQUIRE(mode >= 0 && mode <= 2 && (mode != 2 || (rate && per_rate > 0)), "low_rank_up: bad mode %d", mode);
+    LLB_REQUIRE(mode >= 0 && mode <= 3 && (mode != 2 || (rate && per_rate > 0)), "low_rank_up: bad mode %d", mode);
     LLB_REQUIRE(R <= 512, "low_rank_up: %d inputs; at most 512 (the first half of a low-rank pair is narrow)", R);
     LLB_REQUIRE(out_dtype == LLB_F32 || out_dtype == LLB_BF16, "low_rank_up: unknown output dtype %d", out_dtype);
     LowRankParams p;
     p.x = x; p.x_stride = x_stride; p.x_off = x_off; p.R = R; p.N = N; p.per_rate = per_rate; p.w = w; p.bias = bias;
-    p.rate = rate; p.out = out; p.mode = mode;
+    p.rate = rate; p.out = out; p.mode = mode; p.inv_tau = inv_tau;
     if (x_dtype == LLB_F32 && w_dtype == LLB_F32) return launch_low_rank<float, float>(p, T, out_dtype, stream);
     if (x_dtype == LLB_BF16 && w_dtype == LLB_BF16) return launch_low_rank<__nv_bfloat16, __nv_bfloat16>(p, T, out_dtype, stream);
     if (x_dtype == LLB_BF16 && w_dtype == LLB_F32) return launch_low_rank<__nv_bfloat16, float>(p, T, out_dtype, stream);
     if (x_dtype == LLB_F32 && w_dtype == LLB_BF16) return launch_low_rank<float, __nv_bfloat16>(p, T, out_dtype, stream);
     return llb_fail("low_rank_up: unknown dtypes %d, %d", x_dtype, w_dtype);
+}
+
+LLB_EXPORT int llb_low_rank_up(const void* x, int x_dtype, long long x_stride, int x_off, int T, int R, const void* w,
+                               int w_dtype, int N, const float* bias, int mode, const float* rate, int per_rate,
+                               void* out, int out_dtype, cudaStream_t stream) {
+    return llb_low_rank_up_tau(x, x_dtype, x_stride, x_off, T, R, w, w_dtype, N, bias, mode, rate, per_rate, 1.0f,
+        out, out_dtype, stream);
 }

@@ -87,6 +87,58 @@ __global__ void __launch_bounds__(256) rmsnorm_add_kernel(const float* __restric
     for (int d = lane; d < D; d += 32) o[d] += xr[d] * inv * llb_to_float(w[d]);
 }
 
+// dst[t, :] += sum_i x[i, t, :] / sqrt(mean(x[i, t, :]^2) + eps) * w[i, :]     n <= NORM_SUM_MAX branches side by side; one block
+// a row, four columns a thread and step where V == 4
+constexpr int NORM_SUM_MAX = 4;
+template <int V>
+__global__ void __launch_bounds__(256) rmsnorm_sum_kernel(const float* __restrict__ x, const float* __restrict__ w, float* __restrict__ dst,
+                                                          int n, long long T, int D, float eps) {
+    __shared__ float part[NORM_SUM_MAX][8];
+    const long long t = blockIdx.x;
+    const int warps = blockDim.x >> 5;
+    for (int i = 0; i < n; ++i) {
+        const float* xr = x + ((long long)i * T + t) * D;
+        float ss = 0.0f;
+        for (int d = threadIdx.x * V; d < D; d += blockDim.x * V) {
+            if (V == 4) {
+                const float4 a = *reinterpret_cast<const float4*>(xr + d);
+                ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+            } else {
+                ss = fmaf(xr[d], xr[d], ss);
+            }
+        }
+        ss = llb_warp_sum(ss);
+        if ((threadIdx.x & 31) == 0) part[i][threadIdx.x >> 5] = ss;
+    }
+    __syncthreads();
+    float inv[NORM_SUM_MAX];
+    for (int i = 0; i < n; ++i) {
+        float ss = 0.0f;
+        for (int k = 0; k < warps; ++k) ss += part[i][k];
+        inv[i] = 1.0f / sqrtf(ss / (float)D + eps);
+    }
+    float* o = dst + t * D;
+    for (int d = threadIdx.x * V; d < D; d += blockDim.x * V) {
+        float acc[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[e] = o[d + e];
+        for (int i = 0; i < n; ++i) {
+            const float* xr = x + ((long long)i * T + t) * D + d;
+            const float* wr = w + (long long)i * D + d;
+#pragma unroll
+            for (int e = 0; e < V; ++e) acc[e] += xr[e] * inv[i] * wr[e];
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[d + e] = acc[e];
+    }
+}
+
+// x[t, d] = (x[t, d] + e[t, d]) + v[d]
+__global__ void add_sum_row_kernel(float* __restrict__ x, const float* __restrict__ e, const float* __restrict__ v, long long n, int D) {
+    const long long stride = (long long)gridDim.x * blockDim.x;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) x[i] = (x[i] + e[i]) + v[i % D];
+}
+
 // y[i] += a * x[i]; optionally the new y once more in bf16
 __global__ void axpy_kernel(const float* __restrict__ x, float* __restrict__ y, __nv_bfloat16* __restrict__ copy, long long n, float a) {
     const long long stride = (long long)gridDim.x * blockDim.x;
@@ -127,6 +179,30 @@ LLB_EXPORT int llb_rmsnorm_add(const float* x, const void* w, int w_dtype, float
         rmsnorm_add_kernel<__nv_bfloat16><<<blocks, threads, 0, stream>>>(x, (const __nv_bfloat16*)w, dst, T, D, eps, scale);
     else return llb_fail("rmsnorm_add: unknown weight dtype %d", w_dtype);
     return llb_check_launch("rmsnorm_add");
+}
+
+// dst [T, D] float += sum over the n branches x [n, T, D] float of rmsnorm(x_i) * w_i, w float [n, D] (a branch's factor in the
+// sum is part of its w).
+LLB_EXPORT int llb_rmsnorm_sum(const float* x, const float* w, float* dst, int n, long long T, int D, float eps,
+                               cudaStream_t stream) {
+    if (T == 0 || n == 0) return 0;
+    LLB_REQUIRE(T > 0 && D > 0 && x && w && dst, "rmsnorm_sum: bad arguments");
+    LLB_REQUIRE(n >= 1 && n <= NORM_SUM_MAX && T < (1ll << 31), "rmsnorm_sum: %d branches; at most %d", n, NORM_SUM_MAX);
+    const bool vec = D % 4 == 0 && (uintptr_t)x % 16 == 0;
+    const int per = vec ? D / 4 : D;
+    const int threads = per <= 64 ? 64 : per <= 128 ? 128 : 256;
+    if (vec) rmsnorm_sum_kernel<4><<<(unsigned)T, threads, 0, stream>>>(x, w, dst, n, T, D, eps);
+    else rmsnorm_sum_kernel<1><<<(unsigned)T, threads, 0, stream>>>(x, w, dst, n, T, D, eps);
+    return llb_check_launch("rmsnorm_sum");
+}
+
+// x [T, D] float = (x + e) + v, e float [T, D], v float [D] for every row.
+LLB_EXPORT int llb_add_sum_row(float* x, const float* e, const float* v, long long T, int D, cudaStream_t stream) {
+    if (T == 0) return 0;
+    LLB_REQUIRE(T > 0 && D > 0 && x && e && v, "add_sum_row: bad arguments");
+    const long long n = T * D;
+    add_sum_row_kernel<<<grid_for(n), 256, 0, stream>>>(x, e, v, n, D);
+    return llb_check_launch("add_sum_row");
 }
 
 // y [n] float += a * x [n] float; copy (bf16 [n] or null) receives the new y as well.

@@ -39,18 +39,27 @@ LLB_EXPORT int llb_embedding(const int* ids, const void* table, int table_dtype,
     return llb_check_launch("embedding");
 }
 
-// The same with out = table[ids] * scale, and `copy` ([T, D] in the table's dtype, or null) receiving the same rows.
-LLB_EXPORT int llb_embedding_scaled(const int* ids, const void* table, int table_dtype, float* out, int T, int D, int V,
-                                    int* err, float scale, void* copy, cudaStream_t stream) {
+// The same with out = table[ids] * scale, and `copy` ([T, D] in copy_dtype: float, or the table's; or null) receiving the same rows.
+LLB_EXPORT int llb_embedding_copied(const int* ids, const void* table, int table_dtype, float* out, int T, int D, int V,
+                                    int* err, float scale, void* copy, int copy_dtype, cudaStream_t stream) {
     if (T == 0) return 0;
     LLB_REQUIRE(T > 0 && D > 0 && V > 0, "embedding: bad sizes T=%d D=%d V=%d", T, D, V);
+    LLB_REQUIRE(!copy || copy_dtype == LLB_F32 || copy_dtype == table_dtype, "embedding: the copy is float or has the table's dtype");
     const int threads = D >= 256 ? 256 : 128;
     if (table_dtype == LLB_F32)
         embedding_kernel<float, float><<<T, threads, 0, stream>>>(ids, (const float*)table, out, D, V, err, scale, (float*)copy);
+    else if (table_dtype == LLB_BF16 && copy_dtype == LLB_F32)
+        embedding_kernel<__nv_bfloat16, float><<<T, threads, 0, stream>>>(ids, (const __nv_bfloat16*)table, out, D, V, err, scale,
+                                                                         (float*)copy);
     else if (table_dtype == LLB_BF16)
         embedding_kernel<__nv_bfloat16, __nv_bfloat16><<<T, threads, 0, stream>>>(ids, (const __nv_bfloat16*)table, out, D, V,
                                                                                  err, scale, (__nv_bfloat16*)copy);
     else
         return llb_fail("embedding: unknown table dtype %d", table_dtype);
     return llb_check_launch("embedding");
+}
+
+LLB_EXPORT int llb_embedding_scaled(const int* ids, const void* table, int table_dtype, float* out, int T, int D, int V,
+                                    int* err, float scale, void* copy, cudaStream_t stream) {
+    return llb_embedding_copied(ids, table, table_dtype, out, T, D, V, err, scale, copy, table_dtype, stream);
 }

@@ -398,7 +398,8 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
 #pragma unroll
                         for (int j = 0; j < 16; ++j) {
                             const int m = c0 + j;
-                            const float val = v[j] + bias;
+                            float val = v[j] + bias;
+                            if (EPI == DEPI_STORE_F32 || EPI == DEPI_RESIDUAL) val *= llb_out_scale(p.glu);
                             if (EPI == DEPI_SWIGLU) {
                                 const float other = __shfl_xor_sync(0xffffffffu, val, 1);   // gate: even rows, up: odd rows
                                 if ((lane & 1) == 0 && m < p.M && n + 1 < p.N)
@@ -591,4 +592,14 @@ LLB_EXPORT int llb_gemm_decode_glu(const void* W, const void* a_bf16, const floa
                             split_k, nullptr, nullptr, 0, 0, 0, 0, 0, nullptr, nullptr, nullptr, acc_scratch,
                             scratch_floats, counters, error_flag, LlbGluArgs{glu_kind, glu_alpha, glu_limit, glu_up_shift},
                             stream);
+}
+
+// The float-store and residual epilogues (bf16 operand, no norm prologue) with every output (bias included) times `scale`.
+LLB_EXPORT int llb_gemm_decode_scaled(const void* W, const void* a_bf16, const float* bias, void* out, float* residual,
+                                      int epilogue, int M, int N, int K, int split_k, float scale, int* error_flag,
+                                      cudaStream_t stream) {
+    LLB_REQUIRE(epilogue == DEPI_STORE_F32 || epilogue == DEPI_RESIDUAL, "gemm_decode_scaled: epilogue %d takes no scale", epilogue);
+    return gemm_decode_impl(W, a_bf16, nullptr, nullptr, nullptr, 0, 0.0f, 0, bias, out, residual, epilogue, M, N, K,
+                            split_k, nullptr, nullptr, 0, 0, 0, 0, 0, nullptr, nullptr, nullptr, nullptr, 0, nullptr,
+                            error_flag, LlbGluArgs{LLB_OUT_SCALE, scale, 0.0f, 0.0f}, stream);
 }

@@ -26,12 +26,14 @@ struct Epilogue {
             if (has1) o[1] = llb_from_float<TO>(llb_act(a1, glu.kind));
         } else if (EPI == LLB_EPI_STORE_F32) {
             float* o = (float*)out + (size_t)m * N + n;
-            o[0] = a0;
-            if (has1) o[1] = a1;
+            const float f = llb_out_scale(glu);
+            o[0] = a0 * f;
+            if (has1) o[1] = a1 * f;
         } else if (EPI == LLB_EPI_RESIDUAL) {
             float* r = residual + (size_t)m * N + n;
-            r[0] += a0;
-            if (has1) r[1] += a1;
+            const float f = llb_out_scale(glu);
+            r[0] = fmaf(a0, f, r[0]);
+            if (has1) r[1] = fmaf(a1, f, r[1]);
         } else {  // SWIGLU: column pair (2j, 2j+1) -> output column j of N/2
             TO* o = (TO*)out + (size_t)m * (N / 2) + (n >> 1);
             o[0] = llb_from_float<TO>(llb_glu(a0, a1, glu.kind, glu.alpha, glu.limit, glu.up_shift));

@@ -92,6 +92,11 @@ __device__ __forceinline__ void epilogue_row(const GemmParams& p, int m, int nb,
             for (int j = 0; j < CHUNK; ++j)
                 if (full || nb + j < p.N) v[j] += p.bias[nb + j];
         }
+        if (EPI == LLB_EPI_STORE_F32 || EPI == LLB_EPI_RESIDUAL) {
+            const float f = llb_out_scale(p.glu);
+#pragma unroll
+            for (int j = 0; j < CHUNK; ++j) v[j] *= f;
+        }
         if (EPI == LLB_EPI_SWIGLU) {
             __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)m * (p.N / 2) + (nb >> 1);
             if (full && (p.N % 16) == 0) {     // 16-byte stores of 8 outputs
@@ -282,6 +287,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                         __float2bfloat16_rn(glu_pair<false>(p.glu, v, other));
                             } else if (m < p.M && n < p.N) {
                                 const size_t idx = (size_t)m * p.N + n;
+                                if (EPI == LLB_EPI_STORE_F32 || EPI == LLB_EPI_RESIDUAL) v *= llb_out_scale(p.glu);
                                 if (EPI == LLB_EPI_STORE) ((__nv_bfloat16*)p.out)[idx] = __float2bfloat16_rn(llb_act(v, p.glu.kind));
                                 else if (EPI == LLB_EPI_STORE_F32) ((float*)p.out)[idx] = v;
                                 else if (gridDim.z == 1) p.residual[idx] += v;
@@ -344,6 +350,9 @@ __device__ __forceinline__ void staged_chunk(const GemmParams& p, const CUtensor
     }
     uint8_t* row = stage + lane * 128;
     if (EPI == LLB_EPI_STORE_F32 || EPI == LLB_EPI_RESIDUAL) {
+        const float f = llb_out_scale(p.glu);
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] *= f;
 #pragma unroll
         for (int c = 0; c < 8; ++c)
             *reinterpret_cast<float4*>(row + ((c ^ (lane & 7)) * 16)) = make_float4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
@@ -1011,7 +1020,8 @@ int dispatch_epi(int epi, const CUtensorMap& ma, const CUtensorMap& mb, const Ge
 // to rounding, and the meeting place is not touched).  error_flag: one int that the kernel
 // raises if a wait inside it ran out of time (the result is then invalid), or null.
 // glu_kind .. glu_up_shift: the gated activation of the GLU epilogue (LLB_GLU_*, see llb_glu); under STORE a kind of LlbAct
-// is a plain activation of every output.
+// is a plain activation of every output; under STORE_F32 and RESIDUAL the kind LLB_OUT_SCALE multiplies every output (bias
+// included) by glu_alpha.
 LLB_EXPORT int llb_gemm_tcgen05_glu(const void* A, const void* W, const float* bias, void* out, float* residual,
                                     int epilogue, int M, int N, int K, int split_k, float* partials, int* counters,
                                     int* error_flag, int glu_kind, float glu_alpha, float glu_limit, float glu_up_shift,

@@ -17,7 +17,7 @@ from . import build as _build
 
 F32, BF16 = 0, 1
 EPI_STORE, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU = 0, 1, 2, 3
-ABI_VERSION = 24
+ABI_VERSION = 25
 
 _lib: Optional[ctypes.CDLL] = None
 
@@ -140,7 +140,7 @@ def current_stream() -> int:
 def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: Optional[torch.Tensor] = None,
               scale: float = 1.0, copy: Optional[torch.Tensor] = None) -> None:
     """out[t,:] = table[ids[t],:] * scale as float.  ids int32 [T], table [V,D], out float32 [T,D]; ``copy`` ([T,D] in
-    the table's dtype) receives the same rows."""
+    the table's dtype or float32) receives the same rows."""
     T, (V, D) = ids.numel(), table.shape
     if out.dtype != torch.float32 or tuple(out.shape) != (T, D):
         raise KernelError(f"embedding: out must be float32 [{T},{D}], got {out.dtype} {tuple(out.shape)}")
@@ -148,10 +148,10 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: Op
         _check(lib().llb_embedding(_i32(ids, "ids"), _ptr(table), _dt(table), _ptr(out), T, D, V,
                                    _i32(err, "err"), _stream()))
         return
-    if copy is not None and (copy.dtype != table.dtype or tuple(copy.shape) != (T, D)):
-        raise KernelError(f"embedding: copy must be {table.dtype} [{T},{D}]")
-    _check(lib().llb_embedding_scaled(_i32(ids, "ids"), _ptr(table), _dt(table), _ptr(out), T, D, V, _i32(err, "err"),
-                                      ctypes.c_float(scale), _ptr(copy), _stream()))
+    if copy is not None and (copy.dtype not in (table.dtype, torch.float32) or tuple(copy.shape) != (T, D)):
+        raise KernelError(f"embedding: copy must be {table.dtype} or float32 [{T},{D}]")
+    _check(lib().llb_embedding_copied(_i32(ids, "ids"), _ptr(table), _dt(table), _ptr(out), T, D, V, _i32(err, "err"),
+                                      ctypes.c_float(scale), _ptr(copy), F32 if copy is None else _dt(copy), _stream()))
 
 
 def cast_add(src: torch.Tensor, dst: torch.Tensor, accumulate: bool = False) -> None:
@@ -239,6 +239,11 @@ def attention_scratch_floats(num_tiles: int, num_heads: int, head_dim: int, bq: 
     return int(lib().llb_attention_scratch_floats(num_tiles, num_heads, head_dim, bq, nsplit))
 
 
+def _check_slopes(slopes: Optional[torch.Tensor], num_heads: int) -> None:
+    if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != num_heads):
+        raise KernelError(f"attention: slopes must be float32 [{num_heads}]")
+
+
 def paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
                          tile_span: torch.Tensor, tile_q0: torch.Tensor, num_tiles: int,
                          span_row: torch.Tensor, span_len: torch.Tensor, span_pos: torch.Tensor,
@@ -246,7 +251,8 @@ def paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                          num_heads: int, num_kv_heads: int, head_dim: int, window: int, scale: float,
                          bq: int, nsplit: int = 1, scratch: Optional[torch.Tensor] = None,
                          v_head_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
-                         v_shared: bool = False, softcap: float = 0.0, v_stride: Optional[int] = None) -> None:
+                         v_shared: bool = False, softcap: float = 0.0, v_stride: Optional[int] = None, keep: int = 0,
+                         slopes: Optional[torch.Tensor] = None) -> None:
     """Attention of every query row of the listed tiles over its request's pages.  ``v_head_dim``: width of a value
     row (and of an output row) when it differs from the keys'; ``v_cache`` may be ``k_cache`` itself (values read out
     of the key rows).  ``sinks`` float32 [num_heads]: ``exp(sinks[h])`` joins head h's softmax denominator once.
@@ -254,7 +260,9 @@ def paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
     so ``out`` [T, num_heads, v_head_dim] holds each head's weights applied to the values of every kv head.  ``out`` may
     be float32 under bfloat16 inputs.  ``softcap`` > 0: a score becomes ``softcap * tanh(score / softcap)`` (sinks are
     not capped).  ``v_stride``: numbers from one value row to the next when it is not ``v_head_dim`` (values that are the
-    first ``v_head_dim`` numbers of the key rows: ``head_dim``)."""
+    first ``v_head_dim`` numbers of the key rows: ``head_dim``).  ``keep``: the first ``keep`` positions stay visible whatever
+    the window says.  ``slopes`` float32 [num_heads]: ``slopes[h] * (query position - key position)`` is taken off head h's
+    scores after the cap."""
     hdv = head_dim if v_head_dim is None else v_head_dim
     if k_cache.dtype != q.dtype or v_cache.dtype != q.dtype or out.dtype not in (q.dtype, torch.float32):
         raise KernelError("attention: q and the caches must share a dtype, out has it or is float32")
@@ -262,17 +270,18 @@ def paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         raise KernelError(f"attention: sinks must be float32 [{num_heads}]")
     if out.numel() != q.shape[0] * num_heads * hdv:
         raise KernelError("attention: out does not fit")
+    _check_slopes(slopes, num_heads)
     if nsplit > 1:
         need = attention_scratch_floats(num_tiles, num_heads, hdv, bq, nsplit)
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"attention: nsplit={nsplit} needs {need} floats of scratch")
-    _check(lib().llb_paged_attention_rows(
+    _check(lib().llb_paged_attention_biased(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _dt(q),
         _i32(tile_span, "tile_span"), _i32(tile_q0, "tile_q0"), num_tiles,
         _i32(span_row, "span_row"), _i32(span_len, "span_len"), _i32(span_pos, "span_pos"),
         _i32(block_table, "block_table"), max_pages, page_size, num_heads, num_kv_heads, head_dim, hdv,
         hdv if v_stride is None else v_stride, _ptr(sinks), window, ctypes.c_float(scale), ctypes.c_float(softcap or 0.0), bq, nsplit, _ptr(scratch), 1 if v_shared else 0,
-        1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, _stream()))
+        1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, keep, _ptr(slopes), _stream()))
 
 
 def _f32(t: Optional[torch.Tensor], what: str) -> Optional[int]:
@@ -299,6 +308,7 @@ def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor
 
 GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH = 0, 1, 2
 ACT_SQUARED_RELU = 16          # a plain activation of the contractions' STORE epilogue, in the place of a GLU kind
+OUT_SCALE = 17                 # the contractions' float store and residual epilogues: every output times alpha
 
 
 def glu_act(x: torch.Tensor, out: torch.Tensor, kind: int, alpha: float = 1.0, limit: float = 0.0,
@@ -365,6 +375,27 @@ def rmsnorm_add(x: torch.Tensor, weight: torch.Tensor, eps: float, dst: torch.Te
         raise KernelError("rmsnorm_add: x and dst must be float32 of one shape, weight one value a column")
     _check(lib().llb_rmsnorm_add(_ptr(x), _ptr(weight), _dt(weight), _ptr(dst), ctypes.c_longlong(T), D,
                                  ctypes.c_float(eps), ctypes.c_float(scale), _stream()))
+
+
+RMSNORM_SUM_MAX = 4          # branches that one rmsnorm_sum takes
+
+
+def rmsnorm_sum(x: torch.Tensor, weight: torch.Tensor, eps: float, dst: torch.Tensor) -> None:
+    """dst += sum_i rmsnorm(x[i]) * weight[i], x float32 [n, T, D], weight float32 [n, D], dst float32 [T, D]: several normed
+    branches joining a float sum in one pass (a branch's factor is part of its weight)."""
+    n, T, D = x.shape
+    if x.dtype != torch.float32 or dst.dtype != torch.float32 or tuple(dst.shape) != (T, D) or tuple(weight.shape) != (n, D):
+        raise KernelError("rmsnorm_sum: x float32 [n, T, D], weight float32 [n, D], dst float32 [T, D]")
+    _check(lib().llb_rmsnorm_sum(_ptr(x), _f32(weight, "weight"), _ptr(dst), n, ctypes.c_longlong(T), D, ctypes.c_float(eps),
+                                 _stream()))
+
+
+def add_sum_row(x: torch.Tensor, e: torch.Tensor, v: torch.Tensor) -> None:
+    """x = (x + e) + v: x and e float32 [T, D], v float32 [D] joins every row."""
+    T, D = x.shape
+    if x.dtype != torch.float32 or e.dtype != torch.float32 or tuple(e.shape) != (T, D) or v.dtype != torch.float32 or v.numel() != D:
+        raise KernelError("add_sum_row: x and e must be float32 [T, D] and v float32 [D]")
+    _check(lib().llb_add_sum_row(_ptr(x), _ptr(e), _ptr(v), ctypes.c_longlong(T), D, _stream()))
 
 
 def axpy(x: torch.Tensor, y: torch.Tensor, a: float, copy: Optional[torch.Tensor] = None) -> None:
@@ -662,6 +693,40 @@ def retention(src: torch.Tensor, q_off: int, k_off: int, v_off: int, span_row: t
                                _stream()))
 
 
+def gated_linear(src: torch.Tensor, q_off: int, k_off: int, v_off: int, g: torch.Tensor, q_scale: float, ctx_spans,
+                 num_heads: int, head_dim: int, v_head_dim: int, state: torch.Tensor, state_off: int, out: torch.Tensor,
+                 pieces=None) -> None:
+    """Gated linear attention over every span of the step (csrc/retention.cu): ``S <- diag(exp(g_t)) S + k v^T``,
+    ``o = S^T (q_scale q)``; q, k [H, dim] and v [H, vdim] are column ranges of ``src`` [T, C], ``g`` float32 [T, H*dim] the
+    logarithms of the decays; a request's ``[H, dim, vdim]`` floats lie ``state_off`` into its slot of ``state``; ``out`` float32
+    [T, H*vdim].  ``pieces`` as :func:`retention` takes them."""
+    T, C = src.shape
+    H, dim, vdim = num_heads, head_dim, v_head_dim
+    if max(q_off, k_off) + H * dim > C or v_off + H * vdim > C:
+        raise KernelError("gated_linear: q, k or v lie outside the columns of src")
+    if g.dtype != torch.float32 or g.numel() != T * H * dim or out.dtype != torch.float32 or out.numel() != T * H * vdim:
+        raise KernelError("gated_linear: g must be float32 [T, H*dim] and out float32 [T, H*vdim]")
+    span_row, span_len, span_pos, span_slot, num_spans = ctx_spans
+    base, stride = _state_base(state)
+    if state_off + H * dim * vdim > stride:
+        raise KernelError("gated_linear: the state does not fit in a slot")
+    if pieces is None:
+        iota = torch.arange(num_spans, dtype=torch.int32, device=src.device)
+        pieces = (iota, torch.zeros_like(iota), iota, num_spans, 1 << 30)
+    item_span, item_c, span_first, num_items, chunk = pieces
+    multi = num_items > num_spans
+    scratch = piece_g = None
+    if multi:
+        scratch = torch.empty(num_items * H * dim * vdim, dtype=torch.float32, device=src.device)
+        piece_g = torch.empty(num_items * H * dim, dtype=torch.float32, device=src.device)
+    _check(lib().llb_gated_linear(_ptr(src), _dt(src), ctypes.c_longlong(C), q_off, k_off, v_off, _ptr(g), ctypes.c_float(q_scale),
+                                  _i32(span_row, "span_row"), _i32(span_len, "span_len"), _i32(span_pos, "span_pos"),
+                                  _i32(span_slot, "span_slot"), num_spans, _i32(item_span, "item_span"),
+                                  _i32(item_c, "item_c"), _i32(span_first, "span_first"), num_items, chunk, 1 if multi else 0,
+                                  H, dim, vdim, base, ctypes.c_longlong(stride), ctypes.c_longlong(state_off), _ptr(scratch),
+                                  _ptr(piece_g), _ptr(out), _stream()))
+
+
 # ---- short convolution, delta rule, routing (csrc/short_conv.cu, csrc/delta_rule.cu, csrc/moe.cu) -------------------------
 CONV_NORMS = {None: 0, "rms": 1, "unit": 2}
 
@@ -837,16 +902,21 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, par
                                       _f32(weight, "weight"), _ptr(out), T, n // parts, parts, ctypes.c_float(eps), _stream()))
 
 
-def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, ctx_spans,
+def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: Optional[torch.Tensor], beta: torch.Tensor, ctx_spans,
                num_heads: int, num_qk_heads: int, head_dim: int, v_head_dim: int, state: torch.Tensor, state_off: int,
-               out: torch.Tensor, blocked: bool = False) -> None:
+               out: torch.Tensor, blocked: bool = False, head_decay=None) -> None:
     """The gated delta rule over every span (csrc/delta_rule.cu).  q, k float32 [T, G*dim]; v float32 [T, H*vdim]; g float32
     [T, H*dim] logarithms of the decay factors; ``beta`` a [T, H] view (rows may be strided) of values before the
     sigmoid; the state [H, dim, vdim] of a request lies ``state_off`` floats into its slot of ``state``; out float32
-    [T, H*vdim].  ``blocked`` walks the spans in blocks of 16 tokens (for steps with long spans), else token by token."""
+    [T, H*vdim].  ``head_decay = (a, dt_bias, rate)`` in the place of ``g``: one decay a head, whose logarithm is ``-rate[h] *
+    softplus(a[t, h] + dt_bias[h])``; ``a`` a [T, H] view like ``beta`` (of one dtype and row stride with it), the others float32
+    [H].  ``blocked`` walks the spans in blocks of 16 tokens (for steps with long spans), else token by token."""
     T = q.shape[0]
     H, G, dim, vdim = num_heads, num_qk_heads, head_dim, v_head_dim
-    for t, n, what in ((q, G * dim, "q"), (k, G * dim, "k"), (v, H * vdim, "v"), (g, H * dim, "g"), (out, H * vdim, "out")):
+    if (g is None) == (head_decay is None):
+        raise KernelError("delta_rule: the decays come from g or from head_decay")
+    for t, n, what in ((q, G * dim, "q"), (k, G * dim, "k"), (v, H * vdim, "v"), (out, H * vdim, "out")) \
+            + (((g, H * dim, "g"),) if g is not None else ()):
         if t.dtype != torch.float32 or t.numel() != T * n:
             raise KernelError(f"delta_rule: {what} must be float32 [{T}, {n}]")
     if beta.dim() != 2 or tuple(beta.shape) != (T, H) or beta.stride(1) != 1 or not beta.is_cuda:
@@ -859,21 +929,32 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tenso
     if blocked:          # what the first kernel leaves for the second: bounded by the step's counts alone
         max_blocks = T // 16 + num_spans
         scratch = torch.empty(int(lib().llb_delta_rule_scratch_floats(max_blocks, H, dim)), dtype=torch.float32, device=q.device)
+    spans = (_i32(span_row, "span_row"), _i32(span_len, "span_len"), _i32(span_pos, "span_pos"), _i32(span_slot, "span_slot"),
+             num_spans, H, G, dim, vdim, base, ctypes.c_longlong(stride), ctypes.c_longlong(state_off),
+             _ptr(out), 1 if blocked else 0, _ptr(scratch), max_blocks, _stream())
+    if head_decay is not None:
+        a, dt_bias, rate = head_decay
+        if a.dim() != 2 or tuple(a.shape) != (T, H) or a.stride() != beta.stride() or a.dtype != beta.dtype or not a.is_cuda:
+            raise KernelError(f"delta_rule: the decays' inputs must be [{T}, {H}] with beta's dtype and strides")
+        if dt_bias.numel() != H or rate.numel() != H:
+            raise KernelError(f"delta_rule: dt_bias and rate hold one number for each of the {H} heads")
+        _check(lib().llb_delta_rule_head(_ptr(q), _ptr(k), _ptr(v), ctypes.c_void_p(a.data_ptr()), _f32(dt_bias, "dt_bias"),
+                                         _f32(rate, "rate"), ctypes.c_void_p(beta.data_ptr()),
+                                         ctypes.c_longlong(beta.stride(0)), _dt(beta), *spans))
+        return
     _check(lib().llb_delta_rule(_ptr(q), _ptr(k), _ptr(v), _ptr(g), ctypes.c_void_p(beta.data_ptr()),
-                                ctypes.c_longlong(beta.stride(0)), _dt(beta), _i32(span_row, "span_row"),
-                                _i32(span_len, "span_len"), _i32(span_pos, "span_pos"), _i32(span_slot, "span_slot"),
-                                num_spans, H, G, dim, vdim, base, ctypes.c_longlong(stride), ctypes.c_longlong(state_off),
-                                _ptr(out), 1 if blocked else 0, _ptr(scratch), max_blocks, _stream()))
+                                ctypes.c_longlong(beta.stride(0)), _dt(beta), *spans))
 
 
-LOW_RANK_MODES = {None: 0, "sigmoid": 1, "log_decay": 2}
+LOW_RANK_MODES = {None: 0, "sigmoid": 1, "log_decay": 2, "log_sigmoid": 3}
 
 
 def low_rank_up(x: torch.Tensor, x_off: int, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                mode=None, rate: Optional[torch.Tensor] = None) -> None:
+                mode=None, rate: Optional[torch.Tensor] = None, multiplier: float = 1.0) -> None:
     """out[t, n] = f(sum_r x[t, x_off + r] * w[n, r] + bias[n]) with float sums: the second half of a low-rank pair,
     read from columns of a fused first projection.  ``mode`` None, ``"sigmoid"`` or ``"log_decay"``:
-    ``-rate[h] * softplus(.)`` (the logarithm of a decay factor) with ``rate`` float32 [H] and n = h * (N / H) + ...;
+    ``-rate[h] * softplus(.)`` (the logarithm of a decay factor) with ``rate`` float32 [H] and n = h * (N / H) + ..., or
+    ``"log_sigmoid"``: ``multiplier * ln(sigmoid(.))``;
     out float32 or bfloat16 [T, N]."""
     T, C = x.shape
     N, R = w.shape
@@ -884,8 +965,9 @@ def low_rank_up(x: torch.Tensor, x_off: int, w: torch.Tensor, out: torch.Tensor,
         if rate is None or N % rate.numel():
             raise KernelError("low_rank_up: the decay mode needs one rate per head")
         per = N // rate.numel()
-    _check(lib().llb_low_rank_up(_ptr(x), _dt(x), ctypes.c_longlong(C), x_off, T, R, _ptr(w), _dt(w), N, _f32(bias, "bias"),
-                                 LOW_RANK_MODES[mode], _f32(rate, "rate"), per, _ptr(out), _dt(out), _stream()))
+    _check(lib().llb_low_rank_up_tau(_ptr(x), _dt(x), ctypes.c_longlong(C), x_off, T, R, _ptr(w), _dt(w), N, _f32(bias, "bias"),
+                                     LOW_RANK_MODES[mode], _f32(rate, "rate"), per, ctypes.c_float(multiplier), _ptr(out),
+                                     _dt(out), _stream()))
 
 
 def moe_route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tensor], top: int, scale: float,
@@ -1102,6 +1184,22 @@ def gemm_decode(w: torch.Tensor, epilogue: int, M: int, *, a: Optional[torch.Ten
         _ptr(scratch[1]) if scratch else ctypes.c_void_p(0), _ptr(async_error_flag(w.device)), _stream()))
 
 
+def gemm_decode_scaled(w: torch.Tensor, epilogue: int, a: torch.Tensor, scale: float, bias: Optional[torch.Tensor] = None,
+                       out: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None, split_k: int = 1) -> None:
+    """:func:`gemm_decode` with DEPI_STORE_F32 or DEPI_RESIDUAL, a bf16 operand and every output (bias included) times ``scale``."""
+    N, K = w.shape
+    M = a.shape[0]
+    if w.dtype != torch.bfloat16 or a.dtype != torch.bfloat16 or tuple(a.shape) != (M, K):
+        raise KernelError("gemm_decode_scaled: bfloat16 a [M,K] and w [N,K]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != N):
+        raise KernelError(f"gemm_decode_scaled: bias must be float32 [{N}]")
+    target = residual if epilogue == DEPI_RESIDUAL else out
+    if target is None or target.dtype != torch.float32 or tuple(target.shape) != (M, N):
+        raise KernelError(f"gemm_decode_scaled: the output must be float32 [{M},{N}]")
+    _check(lib().llb_gemm_decode_scaled(_ptr(w), _ptr(a), _ptr(bias), _ptr(out), _ptr(residual), epilogue, M, N, K, split_k,
+                                        ctypes.c_float(scale), _ptr(async_error_flag(w.device)), _stream()))
+
+
 def gemm_decode_glu(w: torch.Tensor, a: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, split_k: int,
                     glu) -> None:
     """The decode contraction's GLU epilogue with the gated activation ``glu`` (as :func:`gemm_simt`): ``a`` bf16 [M, K],
@@ -1133,13 +1231,15 @@ def paged_attention_tcgen05(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
                             span_row: torch.Tensor, span_len: torch.Tensor, span_pos: torch.Tensor,
                             block_table: torch.Tensor, max_pages: int, page_size: int,
                             num_heads: int, num_kv_heads: int, head_dim: int, window: int, scale: float,
-                            cut=None, sinks: Optional[torch.Tensor] = None, cross: int = 1, softcap: float = 0.0) -> None:
+                            cut=None, sinks: Optional[torch.Tensor] = None, cross: int = 1, softcap: float = 0.0,
+                            keep: int = 0, slopes: Optional[torch.Tensor] = None) -> None:
     """Tensor-core attention of the listed tiles (128 query rows each) over the requests' pages; bf16.
     ``sinks`` float32 [num_heads]: ``exp(sinks[h])`` joins head h's softmax denominator once; ``v_cache`` may be
     ``k_cache`` itself (values read out of the key rows).  ``cross`` = ``num_kv_heads`` (> 1): crossed values, ``out``
     is [T, num_heads, cross, head_dim] and holds every query head's weights applied to the values of every kv
     head; ``cut`` must then have been made for ``num_heads * cross`` heads.  ``out`` may be float32.  ``softcap`` > 0: a
-    score becomes ``softcap * tanh(score / softcap)`` before the softmax.
+    score becomes ``softcap * tanh(score / softcap)`` before the softmax.  ``keep`` and ``slopes`` as
+    :func:`paged_attention_simt` (``cut`` must have been made with the same ``keep``).
 
     ``cut`` = ``(tile_k0, tile_nk, tile_part, num_parts, merge_span, merge_q0, merge_first, merge_count,
     num_merge)`` cuts long key ranges into items (see ``StepContext.attention_items``); the partial results
@@ -1161,13 +1261,14 @@ def paged_attention_tcgen05(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
                                   device=q.device)
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != num_heads):
         raise KernelError(f"attention_tcgen05: sinks must be float32 [{num_heads}]")
-    _check(lib().llb_paged_attention_tcgen05_capped(
+    _check_slopes(slopes, num_heads)
+    _check(lib().llb_paged_attention_tcgen05_biased(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), T,
         _i32(tile_span, "tile_span"), _i32(tile_q0, "tile_q0"), num_tiles,
         _i32(span_row, "span_row"), _i32(span_len, "span_len"), _i32(span_pos, "span_pos"),
         _i32(block_table, "block_table"), max_pages, page_size, num_slots, num_heads, num_kv_heads, head_dim,
         window, ctypes.c_float(scale), ctypes.c_float(softcap or 0.0), _i32(k0, "tile_k0"), _i32(nk, "tile_nk"), _i32(part, "tile_part"),
-        _ptr(scratch), num_parts, _ptr(sinks), cross, out_float, _ptr(async_error_flag(q.device)), _stream()))
+        _ptr(scratch), num_parts, _ptr(sinks), cross, out_float, _ptr(async_error_flag(q.device)), keep, _ptr(slopes), _stream()))
     if cut is not None and num_parts:
         _check(lib().llb_attention_tcgen05_merge_cross(
             _ptr(out), _i32(cut[4], "merge_span"), _i32(cut[5], "merge_q0"), _i32(cut[6], "merge_first"),
@@ -1210,11 +1311,13 @@ def paged_decode_mma(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      span_pos: torch.Tensor, block_table: torch.Tensor, max_pages: int, page_size: int,
                      num_heads: int, num_kv_heads: int, head_dim: int, window: int, scale: float,
                      nsplit: int = 1, scratch: Optional[torch.Tensor] = None,
-                     sinks: Optional[torch.Tensor] = None, cross: int = 1, softcap: float = 0.0) -> None:
+                     sinks: Optional[torch.Tensor] = None, cross: int = 1, softcap: float = 0.0, keep: int = 0,
+                     slopes: Optional[torch.Tensor] = None) -> None:
     """Tensor-core decode attention: one query row per tile over its request's pages; bf16.  ``nsplit`` cuts
     each request's keys; up to :func:`decode_mma_cluster_splits` the pieces are merged inside the kernel.
-    ``sinks``, ``v_cache is k_cache``, ``cross`` (crossed values), ``softcap`` and a float32 ``out`` as
+    ``sinks``, ``v_cache is k_cache``, ``cross`` (crossed values), ``softcap``, ``keep``, ``slopes`` and a float32 ``out`` as
     :func:`paged_attention_tcgen05`."""
+    _check_slopes(slopes, num_heads)
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != num_heads):
         raise KernelError(f"decode attention: sinks must be float32 [{num_heads}]")
     for t in (q, k_cache, v_cache):
@@ -1226,12 +1329,12 @@ def paged_decode_mma(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         need = attention_scratch_floats(num_tiles, num_heads * cross, head_dim, 1, nsplit)
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"decode attention: nsplit={nsplit} needs {need} floats of scratch")
-    _check(lib().llb_paged_decode_mma_capped(
+    _check(lib().llb_paged_decode_mma_biased(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _i32(tile_span, "tile_span"), _i32(tile_q0, "tile_q0"),
         num_tiles, _i32(span_row, "span_row"), _i32(span_pos, "span_pos"), _i32(block_table, "block_table"),
         max_pages, page_size, num_heads, num_kv_heads, head_dim, window, ctypes.c_float(scale),
         ctypes.c_float(softcap or 0.0), nsplit,
-        _ptr(scratch), _ptr(sinks), cross, 1 if out.dtype == torch.float32 else 0, _stream()))
+        _ptr(scratch), _ptr(sinks), cross, 1 if out.dtype == torch.float32 else 0, keep, _ptr(slopes), _stream()))
 
 
 # Where the blocks that share a long row of logits meet (a 64-bit slot and a counter per row), per device.

@@ -226,15 +226,17 @@ class StepContext:
         return hit
 
     def attention_items(self, min_len: int, window: int, chunk_tiles: Optional[int] = 4, heads: int = 1,
-                        slots: int = 1, select: Optional[tuple] = None):
+                        slots: int = 1, select: Optional[tuple] = None, keep: int = 0):
         """Work items of the tensor-core attention kernel for the spans of at least ``min_len`` rows: tiles
         of 128 query rows whose key range (in tiles of 128 keys) is cut into pieces of ``chunk_tiles``, longest
         first, so that a long prompt's last rows do not set the kernel's time.  With ``chunk_tiles=None`` the
         piece is as long as the work allows: the tiles of all ``heads`` spread over ``slots`` resident blocks give
         each block so many tiles anyway, and shorter pieces would only add partial results to merge (see
-        :func:`cut_attention_rows`).  ``select`` names the spans by index instead of all of at least ``min_len`` rows.  Returns
+        :func:`cut_attention_rows`).  ``select`` names the spans by index instead of all of at least ``min_len`` rows.  ``keep``: the
+        first ``keep`` positions stay visible beside the window; the key tiles that hold them and lie before the window's first
+        tile count in front of the window's.  Returns
         ``(tile_span, tile_q0, count, cut)`` with ``cut`` as ``ops.paged_attention_tcgen05`` takes it."""
-        key = ("items", min_len, window, chunk_tiles, heads, slots, select)
+        key = ("items", min_len, window, chunk_tiles, heads, slots, select, keep)
         hit = self._tiles.get(key)
         if hit is not None:
             return hit
@@ -248,7 +250,7 @@ class StepContext:
                 pos0 = s.start + q0
                 hi = pos0 + 128 if q0 + 128 <= s.length else s.start + s.length
                 lo = first_visible(pos0, window)
-                rows.append((i, q0, -(-(hi - (lo // 128) * 128) // 128)))
+                rows.append((i, q0, min(-(-keep // 128), lo // 128) + -(-(hi - (lo // 128) * 128) // 128)))
         items, merges, parts = cut_attention_rows(rows, chunk_tiles, heads, slots)
         if not items:
             hit = (self.iota, self.zeros, 0, None)

@@ -59,6 +59,8 @@ class Model:
         for p in self.parts():
             if not isinstance(p, Block):
                 p.bind(tensors, dtype, device)
+        for p in self.parts():
+            p.bound()
 
     def prepare(self, ctx, views) -> None:
         """Every part's ``prepare`` for this step, run entry by run entry (before the metadata copy)."""

@@ -3,8 +3,9 @@ from .base import CacheView, FeedForward, Mixer, Norm, Part, PositionEncoding
 from .attention import AttentionMixer
 from .block import Block, build_part
 from .conv_attention import ConvAttentionMixer
-from .delta import ChannelDeltaMixer
+from .delta import ChannelDeltaMixer, HeadDeltaMixer
 from .differential_attention import DifferentialAttentionMixer
+from .distance_attention import DistanceAttentionMixer
 from .sink_attention import KeyValuedAttentionMixer
 from .moe import RoutedExperts
 from .stream import StreamReinjection, StreamStepVector
@@ -17,6 +18,7 @@ from .gated_attention import GatedAttentionMixer, LatentAttentionMixer
 from .mlp import GatedMLP, PlainMLP
 from .norm import LayerNorm, RMSNorm
 from .retention import RetentionMixer
+from .gated_linear import GatedLinearMixer
 from .rotary_latent_attention import RotaryLatentAttentionMixer
 from .state_space import StateSpaceMixer
 from .rotary import NoPositionEncoding, RotaryEmbedding
@@ -26,4 +28,5 @@ __all__ = ["CacheView", "FeedForward", "Mixer", "Norm", "Part", "PositionEncodin
            "LatentAttentionMixer", "RetentionMixer", "NoPositionEncoding", "RotaryEmbedding", "ConvAttentionMixer",
            "ChannelDeltaMixer", "RoutedExperts", "StreamReinjection", "StreamStepVector", "CausalInputConv",
            "MixedHeadsAttention", "MatrixMemoryMixer", "JoinedMixers", "DifferentialAttentionMixer",
-           "KeyValuedAttentionMixer", "TokenShift", "PlainMLP", "RotaryLatentAttentionMixer", "StateSpaceMixer"]
+           "KeyValuedAttentionMixer", "TokenShift", "PlainMLP", "RotaryLatentAttentionMixer", "StateSpaceMixer",
+           "HeadDeltaMixer", "DistanceAttentionMixer", "GatedLinearMixer"]

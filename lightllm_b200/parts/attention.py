@@ -41,7 +41,8 @@ class AttentionMixer(Mixer):
     q/k/v biases are loaded and added, a token sees its own key, every portion is causal, and
     ``window`` limits a query to the latest ``window`` keys (itself included); ``chunk`` to the keys of its own block
     of ``chunk`` positions, blocks counted from position 0 of the sequence (the kernels take the two as one signed
-    argument: a positive window, or minus the chunk)."""
+    argument: a positive window, or minus the chunk).  ``keep_first``: beside the window the first ``keep_first`` positions
+    of the sequence stay visible."""
 
     graph_safe = True
     takes_rotary_magnitude = False          # whether the mixer's rotation applies the position encoding's `magnitude`
@@ -50,7 +51,10 @@ class AttentionMixer(Mixer):
                  position: Optional[PartSpec] = None, qkv_bias: bool = True, out_bias: bool = False,
                  window: Optional[int] = None, scale: Optional[float] = None,
                  names: Optional[Dict[str, str]] = None, weight_suffix: str = ".weight",
-                 v_head_dim: Optional[int] = None, chunk: Optional[int] = None, cache_window: Optional[int] = None):
+                 v_head_dim: Optional[int] = None, chunk: Optional[int] = None, cache_window: Optional[int] = None,
+                 keep_first: int = 0):
+        if keep_first < 0 or (keep_first and chunk):
+            raise ValueError(f"the first positions are kept beside a window, not beside chunks (keep_first={keep_first})")
         if window and chunk:
             raise ValueError("an attention mixer takes a window or a chunk, not both")
         if num_heads % num_kv_heads:
@@ -71,12 +75,16 @@ class AttentionMixer(Mixer):
         # A soft cap on the scores (set by mixers that have one): score <- softcap * tanh(score / softcap) before the
         # softmax; sinks are not capped.
         self.softcap: Optional[float] = None
+        # A bias by distance (float32 [heads], set by mixers that have one): slopes[h] * (query position - key position) is
+        # taken off head h's (capped) scores; sinks carry none.
+        self.slopes: Optional[torch.Tensor] = None
         self.weight_suffix = weight_suffix
         self.window = window
         # How many of the latest keys the cache plane keeps, when other run entries read this one's plane through windows
         # of their own (0: every key); ``None``: what this mixer's own window needs.
         self.cache_window = cache_window
         self.chunk = int(chunk) if chunk else None
+        self.keep_first = int(keep_first) if window else 0          # without a window nothing needs keeping
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(head_dim)
         self.names = {"q": "q_proj", "k": "k_proj", "v": "v_proj", "o": "o_proj"}
         self.names.update(names or {})
@@ -98,7 +106,7 @@ class AttentionMixer(Mixer):
     def cache_spec(self) -> CacheSpec:
         vd = 0 if self.values_in_keys else (None if self.v_head_dim == self.head_dim else self.v_head_dim)
         keep = self.window if self.cache_window is None else (self.cache_window or None)
-        return CacheSpec(kv=KVSpec(self.num_kv_heads, self.head_dim, keep, vd, self.chunk))
+        return CacheSpec(kv=KVSpec(self.num_kv_heads, self.head_dim, keep, vd, self.chunk, self.keep_first if keep else 0))
 
     def kernel_window(self) -> int:
         """The mask as the attention kernels take it: a window > 0, minus the chunk, or 0 for every earlier key."""
@@ -234,7 +242,8 @@ class AttentionMixer(Mixer):
         # the tensor-core kernels take values as wide as the keys (sinks and values in the key rows included)
         plain = self.v_head_dim == self.head_dim
         cross = self.value_cross
-        key = ("attention_plan", self.num_heads, self.num_kv_heads, self.head_dim, window, dtype, plain, cross)
+        keep = self.keep_first
+        key = ("attention_plan", self.num_heads, self.num_kv_heads, self.head_dim, window, dtype, plain, cross, keep)
         plan = ctx.memo.get(key)
         if plan is not None:
             return plan
@@ -242,7 +251,7 @@ class AttentionMixer(Mixer):
         if ctx.decode_only:
             S = ctx.num_spans
             bound = ctx.max_pages * ctx.page_size          # the same for every step of this shape
-            span = bound if window == 0 else min(bound, abs(window))
+            span = bound if window == 0 else min(bound, abs(window) + keep)
             mma = bf16 and ops.paged_decode_mma_supports(self.num_heads, self.num_kv_heads, self.head_dim)
             # blocks to fill the SMs twice (the tensor-core kernel runs a block per pair of kv heads when values cross)
             want = max(1, -(-2 * L.num_sms(ctx.device) // (S * self.num_kv_heads * (cross if mma else 1))))
@@ -271,7 +280,7 @@ class AttentionMixer(Mixer):
         tensor, single, rows, rest = [], [], [], []
         rows_keys = 0
         for i, s in enumerate(ctx.spans):
-            keys = s.start + s.length if window == 0 else min(s.start + s.length, abs(window) + s.length)
+            keys = s.start + s.length if window == 0 else min(s.start + s.length, abs(window) + self.keep_first + s.length)
             if tc_ok and s.length >= TENSOR_CORE_MIN_ROWS:
                 tensor.append(i)
             elif mma_ok and s.length == 1:
@@ -286,11 +295,11 @@ class AttentionMixer(Mixer):
             blocks_per_sm = 2 if self.head_dim <= 64 else 1
             items = ctx.attention_items(1, window, None, self.num_heads * self.value_cross,
                                         blocks_per_sm * L.num_sms(ctx.device),
-                                        select=tuple(tensor))
+                                        select=tuple(tensor), keep=self.keep_first)
         decode = None
         if single:
             bound = ctx.max_pages * ctx.page_size
-            span = bound if window == 0 else min(bound, abs(window))
+            span = bound if window == 0 else min(bound, abs(window) + self.keep_first)
             resident = (ops.decode_mma_resident(self.head_dim) * L.num_sms(ctx.device)
                         // (len(single) * self.num_kv_heads * self.value_cross))
             nsplit = max(1, min(8, ops.decode_mma_cluster_splits(), resident, -(-span // 128)))
@@ -313,7 +322,7 @@ class AttentionMixer(Mixer):
             if pos_key is None:
                 return None
         return ("attention", self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, self.kernel_window(),
-                self.sinks is not None, self.values_in_keys, self.value_cross, bool(self.softcap), pos_key)
+                self.sinks is not None, self.values_in_keys, self.value_cross, bool(self.softcap), self.keep_first, pos_key)
 
     def prepare(self, ctx, cache=None) -> None:
         self._plan(ctx, ctx.dtype)
@@ -340,7 +349,8 @@ class AttentionMixer(Mixer):
             ops.paged_decode_mma(q, cache.k, v_plane, out, tile_span, tile_q0, ntiles, ctx.span_row, ctx.span_pos,
                                  ctx.block_tables[g], ctx.max_pages, ctx.page_size, self.num_heads,
                                  self.num_kv_heads, self.head_dim, window, self.scale, nsplit, scratch, sinks=self.sinks,
-                                 cross=self.value_cross, softcap=self.softcap or 0.0)
+                                 cross=self.value_cross, softcap=self.softcap or 0.0, keep=self.keep_first,
+                                 slopes=self.slopes)
         elif plan[0] == "decode_simt":
             self._simt(q, cache, out, plan[1], common, 1, plan[2])
         else:
@@ -348,13 +358,15 @@ class AttentionMixer(Mixer):
             if items is not None:
                 tile_span, tile_q0, ntiles, cut = items
                 ops.paged_attention_tcgen05(q, cache.k, v_plane, out, tile_span, tile_q0, ntiles, *common, cut=cut,
-                                            sinks=self.sinks, cross=self.value_cross, softcap=self.softcap or 0.0)
+                                            sinks=self.sinks, cross=self.value_cross, softcap=self.softcap or 0.0, keep=self.keep_first,
+                                 slopes=self.slopes)
             if decode is not None:
                 (tile_span, tile_q0, ntiles), nsplit = decode
                 ops.paged_decode_mma(q, cache.k, v_plane, out, tile_span, tile_q0, ntiles, ctx.span_row, ctx.span_pos,
                                      ctx.block_tables[g], ctx.max_pages, ctx.page_size, self.num_heads,
                                      self.num_kv_heads, self.head_dim, window, self.scale, nsplit, None, sinks=self.sinks,
-                                     cross=self.value_cross, softcap=self.softcap or 0.0)
+                                     cross=self.value_cross, softcap=self.softcap or 0.0, keep=self.keep_first,
+                                 slopes=self.slopes)
             for tiles, bq, nsplit in simt:
                 self._simt(q, cache, out, tiles, common, bq, nsplit)
 
@@ -368,7 +380,8 @@ class AttentionMixer(Mixer):
         ops.paged_attention_simt(q, cache.k, cache.k if self.values_in_keys else cache.v, out, tile_span, tile_q0, ntiles,
                                  *common, bq, nsplit, scratch, v_head_dim=hdv, sinks=self.sinks,
                                  v_shared=self.value_cross > 1, softcap=self.softcap or 0.0,
-                                 v_stride=self.head_dim if self.values_in_keys else None)
+                                 v_stride=self.head_dim if self.values_in_keys else None, keep=self.keep_first,
+                                 slopes=self.slopes)
 
 
 register_part("mixer", "attention", AttentionMixer)

@@ -50,6 +50,9 @@ class Part:
     def bind(self, tensors: Dict[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> None:
         """Take this part's tensors out of ``tensors`` (by the names it declared)."""
 
+    def bound(self) -> None:
+        """Called once when every part of the model has its tensors: the place for what a part makes of its children's."""
+
     def children(self) -> List["Part"]:
         return []
 
@@ -120,6 +123,22 @@ class CacheView:
 
 class Mixer(Part):
     role = "mixer"
+    # True: the output projection multiplies what it adds by ``out_scale`` (a mixer that is one term of a weighted sum).
+    takes_out_scale = False
+    out_scale = 1.0
+
+    def input_weight(self) -> Optional[torch.Tensor]:
+        """The one matrix that reads x, for a mixer whose first kernel is a contraction without a bias and which can run from
+        its result (:meth:`forward_from`): mixers that read one x may then share one contraction.  ``None``: it cannot."""
+        return None
+
+    def share_input(self) -> None:
+        """The owner has taken :meth:`input_weight` into a matrix of its own; this mixer now only runs through
+        :meth:`forward_from`."""
+
+    def forward_from(self, fused, offset: int, residual, ctx, cache) -> None:
+        """:meth:`forward` from ``fused`` [T, C] whose columns from ``offset`` on are ``x @ input_weight()^T``."""
+        raise NotImplementedError
 
     def cache_spec(self) -> Optional[CacheSpec]:
         return None

@@ -90,11 +90,13 @@ _DECODE_EPI = {STORE_F32: ops.DEPI_STORE_F32, RESIDUAL: ops.DEPI_RESIDUAL, SWIGL
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, epilogue: int = STORE,
-           out: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None, glu=None) -> Optional[torch.Tensor]:
+           out: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None, glu=None,
+           scale: float = 1.0) -> Optional[torch.Tensor]:
     """Run the contraction; returns ``out`` (allocated here when not given), or ``None`` for the
     residual epilogue, which adds into ``residual``.  ``glu = (kind, alpha, limit, up_shift)``: the gated activation
     of the SWIGLU epilogue when it is not SiLU (``ops.glu_act`` has the kinds); under STORE a plain activation of every output
-    (``ops.ACT_SQUARED_RELU``)."""
+    (``ops.ACT_SQUARED_RELU``).  ``scale`` (STORE_F32 and RESIDUAL): every output, bias included, is multiplied by it in the
+    epilogue."""
     M, N = x.shape[0], w.shape[0]
     if epilogue != RESIDUAL and out is None:
         cols = N // 2 if epilogue == SWIGLU else N
@@ -102,6 +104,10 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         out = torch.empty((M, cols), dtype=dt, device=x.device)
     if M == 0:
         return out
+    if scale != 1.0:
+        if epilogue not in (STORE_F32, RESIDUAL) or glu is not None:
+            raise ops.KernelError("a scale on the outputs belongs to the float store and residual epilogues")
+        glu = (ops.OUT_SCALE, scale, 0.0, 0.0)
 
     if epilogue in _DECODE_EPI and decode_eligible(M, w, x.dtype, False, _DECODE_EPI[epilogue]):
         split_k = 1
@@ -111,6 +117,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
             split_k = split_k_fused(M, N, x.shape[1])
         if epilogue == SWIGLU and glu is not None:
             ops.gemm_decode_glu(w, x, bias, out, split_k, glu)
+        elif scale != 1.0:
+            ops.gemm_decode_scaled(w, _DECODE_EPI[epilogue], x, scale, bias=bias, out=out, residual=residual, split_k=split_k)
         else:
             ops.gemm_decode(w, _DECODE_EPI[epilogue], M, a=x, bias=bias, out=out, residual=residual, split_k=split_k)
     elif tensor_core_eligible(x, w):

@@ -10,7 +10,7 @@ from ..csrc import ops
 from ..weights import WeightSpec
 from . import linear as L
 from .base import Part
-from .embedding import EMBEDDING_OUTPUT
+from .embedding import EMBEDDING_OUTPUT, EMBEDDING_OUTPUT_F32
 
 
 class StreamReinjection(Part):
@@ -56,16 +56,18 @@ register_part("stream", "reinjection", StreamReinjection)
 
 class StreamStepVector(Part):
     """``h <- h + step[index]``: a learned vector is added to every row of the stream, e.g. before every pass of a looped
-    stretch of layers.  ``step_name`` is ``[steps, hidden]`` and ``index`` picks the row; the sum is float32."""
+    stretch of layers.  ``step_name`` is ``[steps, hidden]`` and ``index`` picks the row.  ``add_embedding``: the embedding
+    output ``e`` (kept in float32 by the embedding part, ``keep_output="float32"``) is added first, ``h <- (h + e) +
+    step[index]``.  The sums are float32, one kernel."""
 
     role = "stream"
     graph_safe = True
 
-    def __init__(self, prefix: str, hidden_size: int, step_name: str, steps: int, index: int):
+    def __init__(self, prefix: str, hidden_size: int, step_name: str, steps: int, index: int, add_embedding: bool = False):
         if not 0 <= index < steps:
             raise ValueError(f"step vector {index} of {steps}")
         self.step_name = f"{prefix}.{step_name}" if prefix else step_name
-        self.hidden_size, self.steps, self.index = hidden_size, steps, index
+        self.hidden_size, self.steps, self.index, self.add_embedding = hidden_size, steps, index, bool(add_embedding)
         self.step = None
 
     def weight_specs(self) -> List[WeightSpec]:
@@ -75,7 +77,13 @@ class StreamStepVector(Part):
         self.step = tensors[self.step_name][self.index].float().contiguous()
 
     def forward(self, residual, ctx) -> None:
-        ops.add_row(residual, self.step)
+        if not self.add_embedding:
+            ops.add_row(residual, self.step)
+            return
+        kept = ctx.memo.get(EMBEDDING_OUTPUT_F32)
+        if kept is None:
+            raise ops.KernelError("step vector: the embedding part did not keep its output in float32 (keep_output='float32')")
+        ops.add_sum_row(residual, kept, self.step)
 
 
 register_part("stream", "step_vector", StreamStepVector)
