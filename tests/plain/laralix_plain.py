@@ -57,24 +57,22 @@ def attention(q, k, v, scale: float, size: Optional[int] = None, keep: int = 0, 
     """q ``[T, H, dim]``, k ``[T, G, dim]``, v ``[T, G, vdim]``; see :func:`visible` for the mask.  ``distance``: the bias of a
     head's slope times the distance is taken off the (capped) score; ``plus_one``: one more in the denominator."""
     T, H, _ = q.shape
-    G = k.shape[1]
+    kv = torch.arange(H) // (H // k.shape[1])                                  # the kv head of every query head
     out = torch.zeros(T, H, v.shape[-1], dtype=q.dtype)
-    slope = slopes(H)
+    slope = torch.tensor(slopes(H), dtype=q.dtype)
     for i in range(T):
         js = torch.tensor([j for j in range(i + 1) if visible(i, j, size, keep)])
-        for h in range(H):
-            g = h // (H // G)
-            s = (k[js, g] @ q[i, h]) * scale
-            if softcap is not None:
-                s = softcap * torch.tanh(s / softcap)
-            if distance:
-                s = s - slope[h] * (i - js).to(q.dtype)
-            m = s.max()
-            if plus_one:
-                m = torch.maximum(m, torch.zeros((), dtype=q.dtype))
-            e = torch.exp(s - m)
-            den = e.sum() + (torch.exp(-m) if plus_one else 0.0)
-            out[i, h] = (e / den) @ v[js, g]
+        s = torch.einsum("hd,jhd->hj", q[i], k[js][:, kv]) * scale
+        if softcap is not None:
+            s = softcap * torch.tanh(s / softcap)
+        if distance:
+            s = s - slope[:, None] * (i - js).to(q.dtype)
+        m = s.max(-1, keepdim=True).values
+        if plus_one:
+            m = torch.clamp(m, min=0.0)
+        e = torch.exp(s - m)
+        den = e.sum(-1, keepdim=True) + (torch.exp(-m) if plus_one else 0.0)
+        out[i] = torch.einsum("hj,jhe->he", e / den, v[js][:, kv])
     return out
 
 
