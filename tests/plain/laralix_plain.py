@@ -53,16 +53,17 @@ def slopes(heads: int) -> List[float]:
 
 
 def attention(q, k, v, scale: float, size: Optional[int] = None, keep: int = 0, softcap: Optional[float] = None,
-              distance: bool = False, plus_one: bool = False) -> torch.Tensor:
-    """q ``[T, H, dim]``, k ``[T, G, dim]``, v ``[T, G, vdim]``; see :func:`visible` for the mask.  ``distance``: the bias of a
+              distance: bool = False, plus_one: bool = False, start: int = 0) -> torch.Tensor:
+    """q ``[T, H, dim]`` (row i at position start + i), k ``[.., G, dim]``, v ``[.., G, vdim]``; see :func:`visible` for the mask.  ``distance``: the bias of a
     head's slope times the distance is taken off the (capped) score; ``plus_one``: one more in the denominator."""
     T, H, _ = q.shape
     kv = torch.arange(H) // (H // k.shape[1])                                  # the kv head of every query head
     out = torch.zeros(T, H, v.shape[-1], dtype=q.dtype)
     slope = torch.tensor(slopes(H), dtype=q.dtype)
-    for i in range(T):
+    for row in range(T):
+        i = start + row
         js = torch.tensor([j for j in range(i + 1) if visible(i, j, size, keep)])
-        s = torch.einsum("hd,jhd->hj", q[i], k[js][:, kv]) * scale
+        s = torch.einsum("hd,jhd->hj", q[row], k[js][:, kv]) * scale
         if softcap is not None:
             s = softcap * torch.tanh(s / softcap)
         if distance:
@@ -72,7 +73,7 @@ def attention(q, k, v, scale: float, size: Optional[int] = None, keep: int = 0, 
             m = torch.clamp(m, min=0.0)
         e = torch.exp(s - m)
         den = e.sum(-1, keepdim=True) + (torch.exp(-m) if plus_one else 0.0)
-        out[i] = torch.einsum("hj,jhe->he", e / den, v[js][:, kv])
+        out[row] = torch.einsum("hj,jhe->he", e / den, v[js][:, kv])
     return out
 
 

@@ -94,6 +94,18 @@ KUTIRAX_BF16_WORST_REL = {"A": 0.0142,           # token by token 0.0141, batch 
                           "A recurrence": 0.0462, "B recurrence": 0.0111, "D recurrence": 0.0075, "E recurrence": 0.0055}
 
 
+# The same for the tiny Laralix configurations of tests/laralix_configs.py (root mean square over a row, as above).
+# C has a width of 32, single heads of 8 and windows of one token: few terms in every norm and softmax.
+LARALIX_BF16_WORST_REL = {"A": 0.0056,           # batch 0.0055, token by token 0.0043, replay 0.0028
+                          "B": 0.0023,           # replay 0.0022
+                          "C": 0.0576,           # replay 0.0575, token by token 0.0473
+                          "D": 0.0060,           # replay 0.0060
+                          "E": 0.0063,           # batch 0.0062, token by token 0.0044, replay 0.0040
+                          "random": 0.0476,      # 0.0476, 0.0279, 0.0190
+                          "A sharp": 0.0025, "B sharp": 0.0023, "D sharp": 0.0041, "E sharp": 0.0035,
+                          "A recurrence": 0.0030, "B recurrence": 0.0021, "D recurrence": 0.0033, "E recurrence": 0.0029}
+
+
 def logits_std(plain_logits) -> float:
     """Standard deviation over all logits of the given plain results (a tensor or a collection of tensors)."""
     if isinstance(plain_logits, torch.Tensor):
