@@ -5,7 +5,7 @@
     python bench.py --sizes 1.5b|7b          (the larger sizes of the family: a line of their own)
     python bench.py [--sizes ..] --only decode|prefill [--prompt-len N]     (one part, at another context length)
     python bench.py --only small-mixed       (the steps of a loaded server: a 16-token portion beside decoded tokens)
-    python bench.py --design kudadra|bulitar|kuzezen|fedirax|kutirax [--sizes 1.5b] [--layers L]     (another design beside Qwen2 at equal sizes)
+    python bench.py --design kudadra|bulitar|kuzezen|fedirax|kutirax|laralix [--sizes 1.5b] [--layers L]     (another design beside Qwen2 at equal sizes)
 
 Prints one JSON line.  ``value`` is decoded tokens a second over K timed decode steps of a
 batch of 8 requests that each hold a 2,048-token prompt (random weights, random token ids),
@@ -440,6 +440,31 @@ def kutirax_config(base: dict, layers: int, kinds=("mamba2", "latent_attention")
                         "mlp": dense if i < dense_first else moe} for i in range(layers)]}
 
 
+def laralix_config(base: dict, layers: int, kinds=("parallel", "parallel_2", "latent_attention")) -> dict:
+    """A Laralix model with the width, feed-forward, head count, head size and vocabulary of a Qwen2 configuration, run as ``layers``
+    layer runs: the first ``layers // 2`` layers twice in a row (the loop), what is left of an odd number once.  Its layers cycle
+    through ``kinds``: distance-biased attention with the base's heads, a cap of 50 and a window of 1,024 beside the delta rule
+    with the base's heads and four taps; attention over a window of 1,024 and the first four tokens beside gated linear attention
+    with the base's heads and a decay rank of 64; latent attention with the base's heads behind a query latent of half the width
+    and a key latent of 256, 32 rotated dimensions."""
+    D, H, G = base["hidden_size"], base["num_attention_heads"], base["num_key_value_heads"]
+    hd = base.get("head_dim", D // H)
+    left = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5}
+    mixers = {
+        "parallel": {"left": {**left, "softcap": 50.0, "mask": {"size": 1024}},
+                     "right": {"heads": H, "kv_heads": H, "dim": hd, "vdim": hd, "conv": 4}},
+        "parallel_2": {"left": {**left, "mask": {"size": 1024, "keep_first": 4}}, "left_scale": 1.1, "right_scale": 0.8,
+                       "right": {"heads": H, "dim": hd, "vdim": hd, "tau": 12.0, "decay_rank": 64}},
+        "latent_attention": {"heads": H, "dim": hd, "rot_dim": 32, "vdim": hd, "q_rank": D // 2, "kv_rank": 256,
+                             "scale": (hd + 32) ** -0.5, "rot": {"dims": 32, "base": 50000.0}},
+    }
+    inner = max(1, layers // 2)
+    return {"architecture": "Laralix", "vocab": base["vocab_size"], "width": D, "embedding": {"scale": 6.0}, "norm": {"eps": 1e-5},
+            "logit_scale": 0.5, "loop": {"start": 0, "stop": inner, "times": 2},
+            "layers": [{"type": kinds[i % len(kinds)], "mixer": mixers[kinds[i % len(kinds)]],
+                        "mlp": {"kind": "dense", "ff": base["intermediate_size"]}} for i in range(inner + max(0, layers - 2 * inner))]}
+
+
 def run_design(name: str, sizes: str, layers: int, steps: int, warmup: int, only=None) -> int:
     """Prefill of one 2,048-token prompt and decode at batch 1 / 8 / 64 over 2,048-token contexts for another design:
     its kinds of layer in turn, each kind alone, and Qwen2 with as many layer runs of the same width, feed-forward,
@@ -466,6 +491,14 @@ def run_design(name: str, sizes: str, layers: int, steps: int, warmup: int, only
                 "kutirax": kutirax_config(base, layers)}
         for kind in ("mamba2", "latent_attention"):
             arms[f"kutirax/{kind}"] = kutirax_config(base, layers, (kind,), dense_first=layers)
+    elif name == "laralix":
+        # beside Qwen2 and the engine's closest designs: Kuzezen (attention beside a recurrence in every layer, looped), Bulitar's
+        # delta rule and Kudadra's retention and latent attention
+        arms = {"qwen2": base, "kuzezen": kuzezen_config(base, layers), "bulitar/channel_delta": bulitar_config(base, layers, ("channel_delta",)),
+                "kudadra/retention": kudadra_config(base, layers, ("retention",)),
+                "kudadra/latent_attention": kudadra_config(base, layers, ("latent_attention",)), "laralix": laralix_config(base, layers)}
+        for kind in ("parallel", "parallel_2", "latent_attention"):
+            arms[f"laralix/{kind}"] = laralix_config(base, layers, (kind,))
     elif name == "kuzezen":
         arms = {"qwen2": base, "kuzezen": kuzezen_config(base, layers),
                 "kuzezen/no feed-forward": kuzezen_config(base, layers, ff=False)}
@@ -509,7 +542,7 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=QWEN25_05B["num_hidden_layers"])
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (for profiling runs)")
-    ap.add_argument("--design", choices=["kudadra", "bulitar", "kuzezen", "fedirax", "kutirax"], default=None,
+    ap.add_argument("--design", choices=["kudadra", "bulitar", "kuzezen", "fedirax", "kutirax", "laralix"], default=None,
                     help="measure another design beside Qwen2 at equal sizes (0.5B sizes, or --sizes; --layers, default 6; "
                          "--only names arms, e.g. kudadra,qwen2): a line of its own, not the bench record")
     ap.add_argument("--sizes", choices=["1.5b", "7b"], default=None,

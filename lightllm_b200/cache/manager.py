@@ -21,7 +21,7 @@ allocated when a device is given.
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Any, Dict, Hashable, List, Optional, Sequence
+from typing import Dict, Hashable, List, Optional, Sequence
 
 import numpy as np
 
@@ -116,8 +116,6 @@ class SeqCache:
     length: int = 0
     tables: List[List[int]] = field(default_factory=list)
     first_live: List[int] = field(default_factory=list)    # first logical page that no window has passed yet
-    version: int = 0                                       # bumped whenever a table changes
-    _np: Dict[int, Any] = field(default_factory=dict)      # group -> (version, int32 array of the table)
 
 
 class CacheManager:
@@ -136,7 +134,14 @@ class CacheManager:
         if len(num_pages) != ngroups:
             raise CacheError(f"num_pages has {len(num_pages)} entries for {ngroups} groups")
         self.pools = [PagePool(n) for n in num_pages]
+        # The groups whose pages are given back while a request lives: (group, window, chunk, logical pages of the first
+        # positions, which stay visible).
+        self._passing = [(g, s.window, s.chunk, -(-s.keep_first // page_size)) for g, s in enumerate(layout.groups)
+                         if s.window is not None or s.chunk]
         self._free_slots: List[int] = list(range(max_seqs - 1, -1, -1))
+        # The live requests' block tables once more, as the step function wants them: per group int32 [max_seqs, pages],
+        # the row of a request's state slot, -1 where it holds no page.
+        self.table_rows = [np.full((max_seqs, self.max_pages_per_seq), -1, dtype=np.int32) for _ in range(ngroups)]
         self.seqs: Dict[Hashable, SeqCache] = {}
         self.dtype = dtype
         self.device = device
@@ -192,14 +197,19 @@ class CacheManager:
         if seq.length + n_tokens > self.max_seq_len:
             raise OutOfPages(f"request {seq_id!r} would hold {seq.length + n_tokens} tokens; "
                              f"the limit is {self.max_seq_len}")
-        needs = self.pages_needed(seq_id, n_tokens)
-        for g, (need, pool) in enumerate(zip(needs, self.pools)):
+        need = max(self.pages_needed(seq_id, n_tokens), default=0)
+        for g, pool in enumerate(self.pools):
             if need > pool.free_count:
                 raise OutOfPages(f"group {g}: {need} pages needed, {pool.free_count} free")
-        for g, (need, pool) in enumerate(zip(needs, self.pools)):
-            if need:
-                seq.tables[g].extend(pool.take_many(seq_id, need))
-                seq.version += 1
+        if need:
+            self._take(seq, need)
+
+    def _take(self, seq: SeqCache, need: int) -> None:
+        """``need`` more pages for a request in every group (they are known to be free)."""
+        for g, pool in enumerate(self.pools):
+            pages, at = pool.take_many(seq.seq_id, need), len(seq.tables[g])
+            seq.tables[g].extend(pages)
+            self.table_rows[g][seq.slot, at: at + need] = pages
 
     def can_reserve_all(self, asks) -> bool:
         """Whether every ``(request, n_tokens)`` of ``asks`` can get its pages at the same time."""
@@ -213,42 +223,45 @@ class CacheManager:
 
     def reserve_all(self, asks) -> None:
         """:meth:`reserve` for several requests at once: all of them get their pages, or none does."""
-        asks = list(asks)
-        if not self.can_reserve_all(asks):
-            for seq_id, n in asks:
-                if self.get(seq_id).length + n > self.max_seq_len:
-                    raise OutOfPages(f"request {seq_id!r} would hold {self.get(seq_id).length + n} tokens; "
-                                     f"the limit is {self.max_seq_len}")
+        needs, total = [], 0          # (a request's tables are equally long in every group)
+        for seq_id, n in asks:
+            seq = self.get(seq_id)
+            held = seq.length + n
+            if held > self.max_seq_len:
+                raise OutOfPages(f"request {seq_id!r} would hold {held} tokens; the limit is {self.max_seq_len}")
+            need = -(-held // self.page_size) - len(seq.tables[0]) if seq.tables else 0
+            if need > 0:
+                needs.append((seq, need))
+                total += need
+        if any(total > pool.free_count for pool in self.pools):
             raise OutOfPages("not enough free pages for this step: free per group "
                              f"{[p.free_count for p in self.pools]}")
-        for seq_id, n in asks:
-            self.reserve(seq_id, n)
+        for seq, need in needs:
+            self._take(seq, need)
 
     def advance(self, seq_id: Hashable, n_tokens: int) -> None:
         """The request now holds ``n_tokens`` more tokens (their keys and values are written).
         Pages that every later query's window has passed are given back."""
         seq = self.get(seq_id)
         new_len = seq.length + n_tokens
-        for g, table in enumerate(seq.tables):
-            if new_len > len(table) * self.page_size:
-                raise CacheError(f"request {seq_id!r} advanced to {new_len} tokens without pages for them")
+        if seq.tables and new_len > len(seq.tables[0]) * self.page_size:
+            raise CacheError(f"request {seq_id!r} advanced to {new_len} tokens without pages for them")
         seq.length = new_len
-        for g, spec in enumerate(self.layout.groups):
-            if spec.window is None and not spec.chunk:
-                continue
+        for g, window, chunk, kept in self._passing:
             first_needed_pos = 0
-            if spec.window is not None:
-                first_needed_pos = new_len - spec.window + 1       # the next query sees keys from here
-            if spec.chunk:                                         # ... and none before its own block of positions
-                first_needed_pos = max(first_needed_pos, new_len - new_len % spec.chunk)
-            dead = max(0, first_needed_pos) // self.page_size   # logical pages wholly before it
+            if window is not None:
+                first_needed_pos = new_len - window + 1            # the next query sees keys from here
+            if chunk:                                              # ... and none before its own block of positions
+                first_needed_pos = max(first_needed_pos, new_len - new_len % chunk)
             table = seq.tables[g]
-            kept = -(-spec.keep_first // self.page_size)           # logical pages of the first positions, which stay visible
-            for lp in range(max(seq.first_live[g], kept), min(dead, len(table))):
+            dead = min(first_needed_pos // self.page_size, len(table))   # logical pages wholly before it
+            if dead <= seq.first_live[g]:
+                continue
+            for lp in range(max(seq.first_live[g], kept), dead):
                 self.pools[g].give(table[lp], seq_id)
                 table[lp] = -1
-                seq.version += 1
-            seq.first_live[g] = max(seq.first_live[g], min(dead, len(table)))
+                self.table_rows[g][seq.slot, lp] = -1
+            seq.first_live[g] = dead
 
     def close(self, seq_id: Hashable) -> None:
         """Give back everything the request holds."""
@@ -257,6 +270,7 @@ class CacheManager:
             for page in table:
                 if page >= 0:
                     self.pools[g].give(page, seq_id)
+            self.table_rows[g][seq.slot, : len(table)] = -1
         self._free_slots.append(seq.slot)
         del self.seqs[seq_id]
 
@@ -277,13 +291,9 @@ class CacheManager:
         return self.get(seq_id).tables[group]
 
     def block_table_array(self, seq_id: Hashable, group: int) -> "np.ndarray":
-        """The block table as an int32 array, rebuilt only when the table has changed."""
+        """The block table as an int32 array (a view: it follows the table)."""
         seq = self.get(seq_id)
-        hit = seq._np.get(group)
-        if hit is None or hit[0] != seq.version:
-            hit = (seq.version, np.asarray(seq.tables[group], dtype=np.int32))
-            seq._np[group] = hit
-        return hit[1]
+        return self.table_rows[group][seq.slot, : len(seq.tables[group])]
 
     def plane_kv(self, group: int, plane: int):
         """(k, v) storage of one plane: ``[pages * page_size, kv_heads, head_dim]`` and ``[..., kv_heads, v_head_dim]``
@@ -322,6 +332,11 @@ class CacheManager:
                                          f"is owned by {pool.owner_of(page)!r}")
             if len(seen) != pool.used_count:
                 raise CacheError(f"group {g}: {pool.used_count} pages in use but {len(seen)} in tables (a page is lost)")
+            rows = np.full_like(self.table_rows[g], -1)
+            for seq in self.seqs.values():
+                rows[seq.slot, : len(seq.tables[g])] = seq.tables[g]
+            if not np.array_equal(rows, self.table_rows[g]):
+                raise CacheError(f"group {g}: the array of block tables differs from the requests' tables")
         slots = [s.slot for s in self.seqs.values()]
         if len(set(slots)) != len(slots) or set(slots) & set(self._free_slots):
             raise CacheError("a state slot is held twice")

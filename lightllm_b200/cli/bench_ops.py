@@ -430,6 +430,64 @@ def main(argv=None) -> int:
     run("moe_route_softmax_over_chosen", lambda: ops.moe_route(x_moe, w_router, None, top, 1.0, r_ids, r_w, r_dense, softmax="chosen",
                                                                bias=rb_s), T * D * 2 + T * E * 4, 2 * T * D * E)
 
+    # ---- one decay a head, a decay a channel and token, a bias by distance, kept first tokens (windows of 1,024) ----------
+    raw_l = rn(T, 2 * Hq, dtype=torch.bfloat16)
+    ones_l, dtb_l = torch.ones(Hq, device=dev), rn(Hq)
+    head = lambda n: (raw_l[:n, Hq:], dtb_l, ones_l)
+    run("delta_rule_head_decay_prompt_in_blocks",
+        lambda: ops.delta_rule(dq, dk, dv, None, raw_l[:, :Hq], spans1, Hq, Hq, hd, hd, conv_state, 0, d_o, blocked=True, head_decay=head(T)),
+        T * Hq * hd * 4 * 4, 8 * T * Hq * hd * hd)
+    run("delta_rule_head_decay_one_token",
+        lambda: ops.delta_rule(dq[:B], dk[:B], dv[:B], None, raw_l[:B, :Hq], spansB, Hq, Hq, hd, hd, conv_state, 0, d_o[:B],
+                               head_decay=head(B)), 2 * B * Hq * hd * hd * 4)
+    run("low_rank_up_log_sigmoid", lambda: ops.low_rank_up(lr_src, 0, w_up, dgate, bias=dt_b, mode="log_sigmoid", multiplier=0.1),
+        T * (rank_lr * 2 + Hq * hd * 4), 2 * T * Hq * hd * rank_lr)
+    gl_state = torch.zeros((B, Hq * hd * hd), device=dev)
+    whole_l = (rB, i32r([0] * B), rB, B, 1 << 30)
+    run("gated_linear_prompt_in_pieces",
+        lambda: ops.gated_linear(ret_src, 0, Hq * hd, 2 * Hq * hd, dgate, hd ** -0.5, spans1, Hq, hd, hd, gl_state, 0, ro,
+                                 pieces=pieces if npieces > 1 else None), T * Hq * hd * (3 * 2 + 4 + 4), 5 * T * Hq * hd * hd)
+    run("gated_linear_one_token",
+        lambda: ops.gated_linear(ret_src[:B], 0, Hq * hd, 2 * Hq * hd, dgate[:B], hd ** -0.5, spansB, Hq, hd, hd, gl_state, 0, roB,
+                                 pieces=whole_l), 2 * B * Hq * hd * hd * 4)
+    two = rn(2, T, D)
+    w_two, dst_two, step_l = rn(2, D), rn(T, D), rn(D)
+    run("rmsnorm_sum_two_branches", lambda: ops.rmsnorm_sum(two, w_two, 1e-5, dst_two), 4 * T * D * 4)
+    run("rmsnorm_add_one_branch", lambda: ops.rmsnorm_add(two[0], w_two[0], 1e-5, dst_two), 3 * T * D * 4)
+    run("add_sum_row", lambda: ops.add_sum_row(dst_two, two[0], step_l), 3 * T * D * 4)
+    nw_l = torch.ones(hd, device=dev)
+    fused_l = rn(T, Nqkv, dtype=torch.bfloat16)
+    run("head_prepare_norm_cache",
+        lambda: ops.head_prepare(fused_l, 0, Hq * hd, Hq, Hkv, hd, positions, positions, q_out, kc, vc, values="columns",
+                                 v_off=(Hq + Hkv) * hd, v_width=Hkv * hd, q_norm_w=nw_l, k_norm_w=nw_l, eps=1e-5), 2 * T * Nqkv * 2)
+    wq_l, wk_l = torch.ones(Hq * hd, device=dev), torch.ones(Hkv * hd, device=dev)
+    run("qkv_prepare_norm_keys_as_values_cache",
+        lambda: ops.qkv_prepare(fused_l, 0, Hq * hd, Hq * hd, Hq, Hkv, hd, hd, positions, positions, q_out, kc, vc, wq_l, wk_l, 1e-5),
+        (T * (Hq + Hkv) * hd + T * Nqkv) * 2)
+    gate_l = rn(T, Hq * hd, dtype=torch.bfloat16)
+    gated_l = torch.empty((T, Hq * hd), dtype=torch.bfloat16, device=dev)
+    run("head_gate_norm_silu", lambda: ops.head_gate(d_o, gate_l, gated_l, Hq, hd, False, "silu", unit_rms=True, eps=1e-5, norm_weight=nw_l),
+        T * Hq * hd * (4 + 2 + 2))
+    slopes_l, zeros_l = torch.tensor([2.0 ** (-8.0 * (h + 1) / Hq) for h in range(Hq)], device=dev), torch.zeros(Hq, device=dev)
+    if ops.attention_tcgen05_supports(hd, page) and T > 128:
+        from lightllm_b200.engine.batch import cut_attention_rows, first_visible
+        from lightllm_b200.parts import linear as L
+        import numpy as np
+        for label, keep_l, kw in (("capped_sinks_bias", 0, dict(sinks=zeros_l, softcap=50.0, slopes=slopes_l)), ("keep_4", 4, dict(keep=4)),
+                                  ("plain", 0, {}), ("capped", 0, dict(softcap=50.0)), ("bias", 0, dict(slopes=slopes_l))):
+            rows_l = [(0, q0, min(-(-keep_l // 128), first_visible(q0, 1024) // 128)
+                       - (-(min(q0 + 128, T) - (first_visible(q0, 1024) // 128) * 128) // 128)) for q0 in range(0, T, 128)]
+            items, merges, parts = cut_attention_rows(rows_l, None, Hq, (2 if hd <= 64 else 1) * L.num_sms(dev))
+            arr = torch.from_numpy(np.asarray([t[1:] for t in items], dtype=np.int32).T.copy()).to(dev)
+            m = torch.from_numpy(np.asarray(merges, dtype=np.int32).reshape(-1, 4).T.copy()).to(dev)
+            cut = (arr[2], arr[3], arr[4], parts, m[0], m[1], m[2], m[3], len(merges)) if merges else (arr[2], arr[3], arr[4], 0, None, None, None, None, 0)
+            keys_seen = sum(min(p + 1, 1024 + keep_l) for p in range(T))
+            ts_l, tq_l = arr[0].contiguous(), arr[1].contiguous()
+            run(f"paged_attention_tcgen05_window_1024_{label}" if label != "plain" else "paged_attention_tcgen05_window_1024",
+                lambda: ops.paged_attention_tcgen05(qp, kcp, vcp, op, ts_l, tq_l, len(items), sr, sl, sp, btp, btp.shape[1], page,
+                                                    Hq, Hkv, hd, 1024, 1 / math.sqrt(hd), cut=cut, **kw),
+                (2 * T * Hq * hd + 2 * T * Hkv * hd) * 2, 2 * 2 * Hq * hd * keys_seen)
+
     # ---- what a decode step of B requests over C keys runs --------------------------------------------------------------
     pages_per = -(-(C + 1) // page)
     kcd = rn(B * pages_per * page, Hkv, hd, dtype=torch.bfloat16)
@@ -448,6 +506,10 @@ def main(argv=None) -> int:
             lambda: ops.paged_decode_mma(qd, kcd, vcd, od, rows, zero, B, rows, pos, btd, pages_per, page, Hq, Hkv, hd, 1024,
                                          1 / math.sqrt(hd), nsplit, None, sinks=sinks_d, softcap=50.0),
             B * min(C + 1, 1024) * Hkv * hd * 2 * 2)
+        for label, kw in (("capped_sinks_bias", dict(sinks=zeros_l, softcap=50.0, slopes=slopes_l)), ("keep_4", dict(keep=4))):
+            run(f"paged_decode_mma_window_1024_{label}",
+                lambda: ops.paged_decode_mma(qd, kcd, vcd, od, rows, zero, B, rows, pos, btd, pages_per, page, Hq, Hkv, hd, 1024,
+                                             1 / math.sqrt(hd), nsplit, None, **kw), B * min(C + 1, 1028) * Hkv * hd * 2 * 2)
         big = 24           # more pieces than a cluster merges: the pieces meet in scratch and a second kernel merges them
         scratch = torch.empty(ops.attention_scratch_floats(B, Hq, hd, 1, big), device=dev)
         run("paged_decode_mma_and_merge", lambda: ops.paged_decode_mma(qd, kcd, vcd, od, rows, zero, B, rows, pos, btd, pages_per,

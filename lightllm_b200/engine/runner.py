@@ -220,21 +220,23 @@ class ModelRunner:
         host[o["span_slot"]: o["span_slot"] + S] = [s.slot for s in spans]
         host[o["iota"]: o["iota"] + S] = np.arange(S, dtype=np.int32)
         host[o["zeros"]: o["zeros"] + S] = 0
-        for g in range(G):
-            bt = host[o["block_tables"] + g * S * P: o["block_tables"] + (g + 1) * S * P].reshape(S, P)
-            sm = host[o["slot_mapping"] + g * T: o["slot_mapping"] + (g + 1) * T]
-            tables_of = {}
-            for i, s in enumerate(spans):
-                table = tables_of.get(s.seq_id)
-                if table is None:
-                    table = tables_of[s.seq_id] = cache.block_table_array(s.seq_id, g)
-                bt[i, : len(table)] = table[:P]
-                bt[i, len(table):] = -1          # "no page": what an earlier step left in the buffer is never an id
-                p = pos[s.row: s.row + s.length]
-                rows = table[p // ps]
-                if rows.min() < 0:
-                    raise StepError(f"request {s.seq_id!r}: a new token falls in a page that was given back")
-                sm[s.row: s.row + s.length] = rows * ps + p % ps
+        if G:
+            # every span's block table and every token's cache row, all spans at once
+            span_slots = np.fromiter((s.slot for s in spans), dtype=np.intp, count=S)
+            lengths = np.fromiter((s.length for s in spans), dtype=np.intp, count=S)
+            token_slots = span_slots if S == T else np.repeat(span_slots, lengths)
+            page_of, in_page = pos // ps, pos % ps
+            for g in range(G):
+                rows = cache.table_rows[g]
+                # (-1 where a request holds no page: what an earlier step left in the buffer is never an id)
+                np.take(rows[:, :P], span_slots, axis=0, mode="clip",
+                        out=host[o["block_tables"] + g * S * P: o["block_tables"] + (g + 1) * S * P].reshape(S, P))
+                pages = rows[token_slots, page_of]
+                if pages.min() < 0:
+                    bad = int(np.argmax(pages < 0))
+                    who = next(s for s in spans if s.row <= bad < s.row + s.length)
+                    raise StepError(f"request {who.seq_id!r}: a new token falls in a page that was given back")
+                np.add(pages * ps, in_page, out=host[o["slot_mapping"] + g * T: o["slot_mapping"] + (g + 1) * T])
         host[o["want_rows"]: o["want_rows"] + R] = want
         if K:
             if min(map_rows) < 0 or max(map_rows) >= T or min(map_from) < 0 or max(map_from) >= token_map[0].numel():
