@@ -133,6 +133,58 @@ __global__ void __launch_bounds__(256) rmsnorm_sum_kernel(const float* __restric
     }
 }
 
+// The same for rows of at most 4 * NV * blockDim.x columns, a multiple of four: every branch's row stays in registers between its
+// sum of squares and the sum.
+template <int NV>
+__global__ void __launch_bounds__(256) rmsnorm_sum_rows_kernel(const float* __restrict__ x, const float* __restrict__ w,
+                                                               float* __restrict__ dst, int n, long long T, int D, float eps) {
+    __shared__ float part[NORM_SUM_MAX][8];
+    const long long t = blockIdx.x;
+    const int warps = blockDim.x >> 5;
+    float4 v[NORM_SUM_MAX][NV], acc[NV];
+    float* o = dst + t * D;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int d = (threadIdx.x + j * blockDim.x) * 4;
+        acc[j] = d < D ? *reinterpret_cast<const float4*>(o + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+#pragma unroll
+    for (int i = 0; i < NORM_SUM_MAX; ++i) {
+        if (i >= n) break;
+        float ss = 0.0f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int d = (threadIdx.x + j * blockDim.x) * 4;
+            const float4 a = d < D ? *reinterpret_cast<const float4*>(x + ((long long)i * T + t) * D + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            v[i][j] = a;
+            ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+        }
+        ss = llb_warp_sum(ss);
+        if ((threadIdx.x & 31) == 0) part[i][threadIdx.x >> 5] = ss;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < NORM_SUM_MAX; ++i) {
+        if (i >= n) break;
+        float ss = 0.0f;
+        for (int k = 0; k < warps; ++k) ss += part[i][k];
+        const float inv = 1.0f / sqrtf(ss / (float)D + eps);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int d = (threadIdx.x + j * blockDim.x) * 4;
+            if (d >= D) continue;
+            const float4 g = *reinterpret_cast<const float4*>(w + (long long)i * D + d);
+            acc[j].x += v[i][j].x * inv * g.x; acc[j].y += v[i][j].y * inv * g.y;
+            acc[j].z += v[i][j].z * inv * g.z; acc[j].w += v[i][j].w * inv * g.w;
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int d = (threadIdx.x + j * blockDim.x) * 4;
+        if (d < D) *reinterpret_cast<float4*>(o + d) = acc[j];
+    }
+}
+
 // x[t, d] = (x[t, d] + e[t, d]) + v[d]
 __global__ void add_sum_row_kernel(float* __restrict__ x, const float* __restrict__ e, const float* __restrict__ v, long long n, int D) {
     const long long stride = (long long)gridDim.x * blockDim.x;
@@ -188,7 +240,13 @@ LLB_EXPORT int llb_rmsnorm_sum(const float* x, const float* w, float* dst, int n
     if (T == 0 || n == 0) return 0;
     LLB_REQUIRE(T > 0 && D > 0 && x && w && dst, "rmsnorm_sum: bad arguments");
     LLB_REQUIRE(n >= 1 && n <= NORM_SUM_MAX && T < (1ll << 31), "rmsnorm_sum: %d branches; at most %d", n, NORM_SUM_MAX);
-    const bool vec = D % 4 == 0 && (uintptr_t)x % 16 == 0;
+    const bool vec = D % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)dst % 16 == 0;
+    if (vec && D <= 2048) {
+        const int quads = D / 4;
+        if (quads <= 256) rmsnorm_sum_rows_kernel<1><<<(unsigned)T, (quads + 31) / 32 * 32, 0, stream>>>(x, w, dst, n, T, D, eps);
+        else rmsnorm_sum_rows_kernel<2><<<(unsigned)T, 256, 0, stream>>>(x, w, dst, n, T, D, eps);
+        return llb_check_launch("rmsnorm_sum");
+    }
     const int per = vec ? D / 4 : D;
     const int threads = per <= 64 ? 64 : per <= 128 ? 128 : 256;
     if (vec) rmsnorm_sum_kernel<4><<<(unsigned)T, threads, 0, stream>>>(x, w, dst, n, T, D, eps);

@@ -320,7 +320,7 @@ def test_log_sigmoid_decays_from_a_low_rank_pair(dtype, T, R, N):
 # ---------------------------------------------------------------------------------------------------------------------
 # small pieces
 # ---------------------------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("n,T,D", [(2, 1, 44), (2, 37, 256), (1, 5, 50), (4, 9, 1030), (3, 300, 64)])
+@pytest.mark.parametrize("n,T,D", [(2, 1, 44), (2, 37, 256), (1, 5, 50), (4, 9, 1030), (3, 300, 64), (2, 40, 1028), (4, 3, 2048), (2, 5, 2052), (2, 7, 896)])
 def test_normed_branches_join_in_one_pass(n, T, D):
     torch.manual_seed(D)
     x, w, dst = torch.randn(n, T, D) * 3, torch.randn(n, D), torch.randn(T, D)
